@@ -1242,7 +1242,7 @@ def tosevik_kernels(a, z, P, B, ctx, pk):
                 res[f"{name}_decode"]["experts_touched"] = touched
         z_ = f32(N, E + 1)
         idc, wtc = torch.empty(N, top, dtype=torch.int32, device=dev), torch.empty(N, top, device=dev)
-        us = timed(lambda: ops.moe_select(z_, None, idc, wtc, z["groups"], z["keep"], experts=E, softmax=True, worth="max", scale=2.5))
+        us = timed(lambda: ops.moe_select(z_, None, idc, wtc, z["groups"], z["keep"], experts=E, score="softmax", worth="max", scale=2.5))
         res[f"choice_softmax_{form}"] = {"us": us}
         corr = f32(E)
         us = timed(lambda: ops.moe_select(z_, corr, idc, wtc, z["groups"], z["keep"], experts=E))

@@ -33,10 +33,12 @@ from .pages import Pool
 class CacheNeed:
     """What one mixer keeps per position: kind "full" (every position), "window" (the last `window` positions) or
     "chunk" (the positions of the query's own block of `window` positions, blocks counted from position 0), and
-    `tensors`, one (heads, width) per tensor a position holds, each stored in a pool of its own."""
+    `tensors`, one (heads, width) per tensor a position holds, each stored in a pool of its own.  keep: behind a window
+    the first `keep` positions of the sequence are still read, so their pages stay until the request ends."""
     kind: str
     tensors: tuple
     window: Optional[int] = None
+    keep: int = 0
 
     def merged(self, other):
         """-> the need that serves both mixers when they share one cache (one writes it, the other reads it), or None
@@ -51,7 +53,7 @@ class CacheNeed:
             if big % small == 0:
                 return CacheNeed("chunk", self.tensors, big)
         if self.kind == other.kind == "window":
-            return CacheNeed("window", self.tensors, max(self.window, other.window))
+            return CacheNeed("window", self.tensors, max(self.window, other.window), max(self.keep, other.keep))
         return CacheNeed("full", self.tensors, None)
 
     @classmethod
@@ -102,7 +104,7 @@ class CacheManager:
             if need is None:
                 continue
             if need.kind not in ("full", "window", "chunk") or (need.kind != "full" and not need.window) \
-                    or not need.tensors \
+                    or not need.tensors or need.keep < 0 or (need.keep and need.kind != "window") \
                     or any(len(t) != 2 or min(t) < 1 for t in need.tensors):
                 raise CacheError(f"cache need {need} is not understood")
             by_need.setdefault(need, []).append(cid)
@@ -130,6 +132,10 @@ class CacheManager:
             for cid, s in self.state_needs.items():
                 self.state[cid] = torch.zeros((self.max_requests + 1,) + tuple(s.shape), dtype=getattr(torch, s.dtype),
                                               device=device)
+
+    def _kept_blocks(self, g):
+        """blocks at the start of a sequence that group g never gives back before the request ends"""
+        return -(-g.need.keep // self.page_size)
 
     # -------------------------------------------------------------------------------------------- requests
     def admit(self, rid):
@@ -205,7 +211,7 @@ class CacheManager:
         r.length += n_new
         for gi, g in enumerate(self.groups):
             first = min(self._first_needed(g, r.length), -(-r.reserved // self.page_size))
-            for b in range(r.first_block[gi], first):
+            for b in range(max(r.first_block[gi], self._kept_blocks(g)), first):
                 pg = int(g.table[r.row, b])
                 if pg >= 0:
                     g.pool.give(pg)
@@ -253,13 +259,13 @@ class CacheManager:
     def pages_to_hold(self, tokens, portion):
         """-> per group, the most pages a request of `tokens` tokens holds at any time when it is fed in portions of at
         most `portion` tokens: every page of a full group; of a window group only those the window and one portion
-        reach (what lies behind the window is given back at every commit); a chunk group likewise, with its block of
+        reach (what lies behind the window is given back at every commit) and those of the kept first positions; a chunk group likewise, with its block of
         positions in the window's place"""
         whole = -(-int(tokens) // self.page_size)
         out = []
         for g in self.groups:
             if g.need.kind in ("window", "chunk"):
-                out.append(min(whole, -(-(g.need.window - 1 + int(portion)) // self.page_size) + 1))
+                out.append(min(whole, -(-(g.need.window - 1 + int(portion)) // self.page_size) + 1 + self._kept_blocks(g)))
             else:
                 out.append(whole)
         return out

@@ -53,12 +53,16 @@ def _builtin():
     if _done:
         return
     _done = True
-    from ..models import fipitar, llama, luzosun, sufopel, tosevik
+    from ..models import fipitar, llama, luzosun, pobelorn, sufopel, tosevik
     from .fipitar import FipitarConfig
     from .llama import LlamaConfig
     from .luzosun import LuzosunConfig
+    from .pobelorn import PobelornConfig
     from .sufopel import SufopelConfig
     from .tosevik import TosevikConfig
+    if "Pobelorn" not in ARCHITECTURES:
+        register_architecture(Architecture("Pobelorn", PobelornConfig, pobelorn.model_spec, pobelorn.canonical_names,
+                                           pobelorn.stored_tensors))
     if "Fipitar" not in ARCHITECTURES:
         register_architecture(Architecture("Fipitar", FipitarConfig, fipitar.model_spec, fipitar.canonical_names,
                                            fipitar.stored_tensors))

@@ -1,7 +1,9 @@
 // Paged flash attention on tensor cores (bf16) in its GENERAL form: keys of GA_DK and values of GA_DV values (the
 // library is compiled for one such pair, -DGA_DK=.. -DGA_DV=..; both multiples of 16 up to 256), pools whose rows may
 // be wider than what is read of them (k_row, v_row: elements between two positions' rows; a pool whose row is key and
-// value at once is handed in twice), and, each optional: capped scores s <- cap tanh(s / cap); a sink per query head,
+// value at once is handed in twice), and, each optional: first positions
+// that stay visible behind a window (`keep`: the key tiles are then those of the kept positions and those of the window,
+// with a gap between); capped scores s <- cap tanh(s / cap); a sink per query head,
 // one more term exp(sink_h) in the softmax's denominator that has no value; a gate per token and query head, the
 // head's result times sigmoid(gate).
 //
@@ -28,6 +30,7 @@ struct GenParams {
     float scale, softcap;                   // softcap 0: none
     const float* sinks;                     // one per query head, or null
     const bf16* gate; int gate_stride;      // gate[n * gate_stride + h], or null
+    int keep;                               // behind the window the first `keep` positions stay visible
 };
 
 // what a finished row is multiplied by and what its denominator gains: the sink joins after every key
@@ -45,7 +48,7 @@ __device__ __forceinline__ void ga_finish(const GenParams& P, int n, int h, floa
 
 template <int HD, int BN>
 __device__ __forceinline__ void load_tile(bf16* dst, const bf16* pool, int row_elems, const AttnParams& P, const int* tb,
-                                          int kvh, int kb, int lo, int hi, int tid) {
+                                          int kvh, int kb, int lo, int hi, int keep, int tid) {
     constexpr int CH = HD / 8;
     const int shift = P.page_shift, mask = P.page - 1;
     int last_block = -1, pg = -1;
@@ -55,7 +58,7 @@ __device__ __forceinline__ void load_tile(bf16* dst, const bf16* pool, int row_e
         const int kp = kb + row;
         const bf16* src = pool;
         int bytes = 0;
-        if (kp >= lo && kp < hi) {                       // below lo a window may have given the pages back
+        if ((kp >= lo || kp < keep) && kp < hi) {        // below lo a window may have given the pages back
             int block, slot;
             if (shift >= 0) { block = kp >> shift; slot = kp & mask; }
             else { block = kp / P.page; slot = kp - block * P.page; }
@@ -99,7 +102,10 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
     const int hi = pos_max + 1;
     const int lo = (P.window > 0 && pos_min - P.window + 1 > 0) ? pos_min - P.window + 1 : 0;
     const int lo_al = (lo / BN) * BN;
-    const int n_tiles = (hi - lo_al + BN - 1) / BN;
+    // with kept first positions: the tiles that hold them, as far as they end before the window's first tile, come first
+    const int front = min((GP.keep + BN - 1) / BN, lo_al / BN), skip = lo_al / BN - front;
+    const int n_tiles = front + (hi - lo_al + BN - 1) / BN;
+    auto tile_key = [&](int t) { return (t < front ? t : t + skip) * BN; };
     const int tps = (n_tiles + n_splits - 1) / n_splits;
     const int t_begin = split * tps, t_end = min(n_tiles, t_begin + tps);
     const int* tb = P.table + (size_t)P.seq_row[seq] * P.max_blocks;
@@ -117,8 +123,8 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
     cp_async_commit();
     auto fetch = [&](int t) {
         bf16* st = kvs + (size_t)((t - t_begin) % STAGES) * STAGE;
-        load_tile<DK, BN>(st, P.kpool, GP.k_row, P, tb, kvh, lo_al + t * BN, lo, hi, tid);
-        if (!SHARED) load_tile<DV, BN>(st + BN * ROWK, P.vpool, GP.v_row, P, tb, kvh, lo_al + t * BN, lo, hi, tid);
+        load_tile<DK, BN>(st, P.kpool, GP.k_row, P, tb, kvh, tile_key(t), lo, hi, GP.keep, tid);
+        if (!SHARED) load_tile<DV, BN>(st + BN * ROWK, P.vpool, GP.v_row, P, tb, kvh, tile_key(t), lo, hi, GP.keep, tid);
     };
 #pragma unroll
     for (int s = 0; s < STAGES - 1; s++) {
@@ -165,7 +171,7 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
         }
         const bf16* kt = kvs + (size_t)((t - t_begin) % STAGES) * STAGE;
         const bf16* vt = SHARED ? kt : kt + BN * ROWK;
-        const int kb = lo_al + t * BN;
+        const int kb = tile_key(t);
 
         float s[NT][4];
 #pragma unroll
@@ -188,7 +194,7 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
             for (int e = 0; e < 4; e++) {
                 const int i = e >> 1;
                 const int key = kb + nbase + j * 8 + 2 * tig + (e & 1);
-                const bool ok = key <= rpos[i] && key >= rlo[i];
+                const bool ok = key <= rpos[i] && (key >= rlo[i] || key < GP.keep);
                 float v = s[j][e] * GP.scale;
                 // tanh(x) = 1 - 2 / (e^2x + 1) on the fast exponential and division (a few ulp; both ends saturate cleanly):
                 // tanhf's own code was the longest chain of the tile (stalls on fixed-latency waits, tensor pipe 20 %)
@@ -363,7 +369,7 @@ static void ga_fill(GenParams& GP, const void* q, int q_stride, void* out, const
                     int v_row, const int* q_start, const int* q_len, const int* pos0, const int* part_base,
                     const int* seq_row, const int* table, int max_blocks, float* part_o, float* part_ml, int max_splits,
                     int H, int KV, int page, int num_pages, int window, float scale, float softcap, const float* sinks,
-                    const void* gate, int gate_stride, int* err) {
+                    const void* gate, int gate_stride, int keep, int* err) {
     AttnParams& P = GP.a;
     P.q = (const bf16*)q; P.q_stride = q_stride; P.out = (bf16*)out;
     P.kpool = (const bf16*)kpool; P.vpool = (const bf16*)vpool;
@@ -378,6 +384,7 @@ static void ga_fill(GenParams& GP, const void* q, int q_stride, void* out, const
     P.err = err;
     GP.k_row = k_row; GP.v_row = v_row; GP.scale = scale; GP.softcap = softcap; GP.sinks = sinks;
     GP.gate = (const bf16*)gate; GP.gate_stride = gate_stride;
+    GP.keep = window > 0 ? keep : 0;        // without a window every position is visible anyway
 }
 
 // decode != 0: items are tiles of at most 16 rows; else tiles of 64 rows.
@@ -386,14 +393,15 @@ MB_API int mb_attn_general_bf16(const void* q, int q_stride, void* out, const vo
                                 const int* q_len, const int* pos0, const int* part_base, const int* seq_row,
                                 const int* table, int max_blocks, float* part_o, float* part_ml, int max_splits, int H,
                                 int KV, int DK, int DV, int page, int num_pages, int window, float scale, float softcap,
-                                const float* sinks, const void* gate, int gate_stride, int* err, cudaStream_t st) {
+                                const float* sinks, const void* gate, int gate_stride, int keep, int* err,
+                                cudaStream_t st) {
     if (n_items == 0) return 0;
-    if (DK != GA_DK || DV != GA_DV || KV < 1 || H % KV || KV > 65535 || k_row < DK || v_row < DV || (k_row & 7) ||
+    if (keep < 0 || DK != GA_DK || DV != GA_DV || KV < 1 || H % KV || KV > 65535 || k_row < DK || v_row < DV || (k_row & 7) ||
         (v_row & 7) || (q_stride & 7))
         return -2;
     GenParams GP;
     ga_fill(GP, q, q_stride, out, kpool, vpool, k_row, v_row, q_start, q_len, pos0, part_base, seq_row, table, max_blocks,
-            part_o, part_ml, max_splits, H, KV, page, num_pages, window, scale, softcap, sinks, gate, gate_stride, err);
+            part_o, part_ml, max_splits, H, KV, page, num_pages, window, scale, softcap, sinks, gate, gate_stride, keep, err);
     GP.a.items = (const int4*)items;
     constexpr int WIDE = (GA_DK > 128 || GA_DV > 128) ? 1 : 0;
     constexpr bool CAN_SHARE = GA_DV <= GA_DK;
@@ -410,7 +418,7 @@ MB_API int mb_attn_general_merge_bf16(float* part_o, float* part_ml, const void*
     if (n_part == 0) return 0;
     GenParams GP;
     ga_fill(GP, nullptr, 0, out, nullptr, nullptr, 0, 0, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, 0, part_o,
-            part_ml, max_splits, H, 1, 1, 0, 0, 1.0f, 0.0f, sinks, gate, gate_stride, nullptr);
+            part_ml, max_splits, H, 1, 1, 0, 0, 1.0f, 0.0f, sinks, gate, gate_stride, 0, nullptr);
     attn_general_merge_kernel<<<dim3(n_part, H), 128, 0, st>>>(GP, (const int2*)part_tok, DV);
     MB_LAUNCH_CHECK();
     return 0;

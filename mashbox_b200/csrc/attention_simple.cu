@@ -7,7 +7,7 @@
 // row of either pool may be wider than what is read of it (k_row, v_row: the distance between two positions' rows; a
 // pool whose rows are key and value at once is handed in twice).  Optional: a cap on the scores, s <- cap tanh(s / cap);
 // a sink per query head, one more term exp(sink_h) in the softmax's denominator that has no value; a gate per token and
-// query head, the head's result times sigmoid(gate).
+// query head, the head's result times sigmoid(gate); behind a window, the first `keep` positions stay visible.
 #include "common.cuh"
 
 #define SIMPLE_MAX_HD 1024         // the widest rows (three instantiations: up to 256, up to 512, and up to this)
@@ -19,7 +19,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_simple_kernel(
     const int* __restrict__ tok_seq, const int* __restrict__ table, int max_blocks, const T* __restrict__ kpool,
     const T* __restrict__ vpool, int N, int H, int KV, int HD, int page, int num_pages, int window, float scale,
     int* err, int HDV, int k_row, int v_row, float softcap, const float* __restrict__ sinks,
-    const T* __restrict__ gate, int gate_stride) {
+    const T* __restrict__ gate, int gate_stride, int keep) {
     __shared__ float qs[WARPS][MAXHD];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * WARPS + warp;
@@ -36,9 +36,11 @@ __global__ void __launch_bounds__(WARPS * 32) attn_simple_kernel(
     float acc[MAXHD / 32];
 #pragma unroll
     for (int i = 0; i < MAXHD / 32; i++) acc[i] = 0.0f;
-    for (int base = lo; base <= pos; base += 32) {
-        const int kp = base + lane;
-        const bool valid = kp <= pos;
+    // the keys that are seen, numbered in ascending order: `front` kept ones, then the window's
+    const int front = min(keep, lo), seen = front + pos - lo + 1;
+    for (int base = 0; base < seen; base += 32) {
+        const int kp = base + lane < front ? base + lane : lo + base + lane - front;
+        const bool valid = base + lane < seen;
         long long off = -1;        // the position's row among the rows of its kv head's pages (times k_row or v_row)
         float s = -INFINITY;
         if (valid) {
@@ -62,7 +64,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_simple_kernel(
         l = l * corr + mb_warp_sum(p);
 #pragma unroll
         for (int i = 0; i < MAXHD / 32; i++) acc[i] *= corr;
-        const int cnt = min(32, pos - base + 1);
+        const int cnt = min(32, seen - base);
         for (int j = 0; j < cnt; j++) {
             const float pj = __shfl_sync(0xffffffffu, p, j);
             const long long oj = __shfl_sync(0xffffffffu, off, j);
@@ -97,27 +99,28 @@ static int attn_simple_launch(const void* q, int q_stride, void* out, const int*
                               const int* table, int max_blocks, const void* kpool, const void* vpool, int N, int H,
                               int KV, int HD, int page, int num_pages, int window, float scale, int* err,
                               cudaStream_t st, int HDV = 0, int k_row = 0, int v_row = 0, float softcap = 0.0f,
-                              const float* sinks = nullptr, const void* gate_ = nullptr, int gate_stride = 0) {
+                              const float* sinks = nullptr, const void* gate_ = nullptr, int gate_stride = 0,
+                              int keep = 0) {
     if (N == 0) return 0;
     if (HDV == 0) HDV = HD;
     if (k_row == 0) k_row = HD;
     if (v_row == 0) v_row = HDV;
     const T* gate = (const T*)gate_;
     const int widest = HD > HDV ? HD : HDV;
-    if (widest > SIMPLE_MAX_HD || HD < 1 || HDV < 1 || KV < 1 || H % KV || k_row < HD || v_row < HDV) return -2;
+    if (widest > SIMPLE_MAX_HD || keep < 0 || HD < 1 || HDV < 1 || KV < 1 || H % KV || k_row < HD || v_row < HDV) return -2;
     const long long items = (long long)N * H;
     if (widest <= 256)
         attn_simple_kernel<T, 256><<<(unsigned)((items + WARPS - 1) / WARPS), WARPS * 32, 0, st>>>(
             (const T*)q, q_stride, (T*)out, positions, tok_seq, table, max_blocks, (const T*)kpool, (const T*)vpool, N, H,
-            KV, HD, page, num_pages, window, scale, err, HDV, k_row, v_row, softcap, sinks, gate, gate_stride);
+            KV, HD, page, num_pages, window, scale, err, HDV, k_row, v_row, softcap, sinks, gate, gate_stride, keep);
     else if (widest <= 512)
         attn_simple_kernel<T, 512><<<(unsigned)((items + WARPS - 1) / WARPS), WARPS * 32, 0, st>>>(
             (const T*)q, q_stride, (T*)out, positions, tok_seq, table, max_blocks, (const T*)kpool, (const T*)vpool, N, H,
-            KV, HD, page, num_pages, window, scale, err, HDV, k_row, v_row, softcap, sinks, gate, gate_stride);
+            KV, HD, page, num_pages, window, scale, err, HDV, k_row, v_row, softcap, sinks, gate, gate_stride, keep);
     else
         attn_simple_kernel<T, SIMPLE_MAX_HD><<<(unsigned)((items + WARPS - 1) / WARPS), WARPS * 32, 0, st>>>(
             (const T*)q, q_stride, (T*)out, positions, tok_seq, table, max_blocks, (const T*)kpool, (const T*)vpool, N, H,
-            KV, HD, page, num_pages, window, scale, err, HDV, k_row, v_row, softcap, sinks, gate, gate_stride);
+            KV, HD, page, num_pages, window, scale, err, HDV, k_row, v_row, softcap, sinks, gate, gate_stride, keep);
     MB_LAUNCH_CHECK();
     return 0;
 }
@@ -141,18 +144,18 @@ MB_API int mb_attn_simple_bf16(const void* q, int q_stride, void* out, const int
 MB_API int mb_attn_simple_ext_f32(const void* q, int q_stride, void* out, const int* positions, const int* tok_seq,
                                   const int* table, int max_blocks, const void* kpool, const void* vpool, int N, int H,
                                   int KV, int HD, int HDV, int k_row, int v_row, int page, int num_pages, int window,
-                                  float scale, float softcap, const float* sinks, const void* gate, int gate_stride,
+                                  float scale, float softcap, const float* sinks, const void* gate, int gate_stride, int keep,
                                   int* err, cudaStream_t st) {
     return attn_simple_launch<float>(q, q_stride, out, positions, tok_seq, table, max_blocks, kpool, vpool, N, H, KV,
                                      HD, page, num_pages, window, scale, err, st, HDV, k_row, v_row, softcap, sinks, gate,
-                                     gate_stride);
+                                     gate_stride, keep);
 }
 MB_API int mb_attn_simple_ext_bf16(const void* q, int q_stride, void* out, const int* positions, const int* tok_seq,
                                    const int* table, int max_blocks, const void* kpool, const void* vpool, int N, int H,
                                    int KV, int HD, int HDV, int k_row, int v_row, int page, int num_pages, int window,
-                                   float scale, float softcap, const float* sinks, const void* gate, int gate_stride,
+                                   float scale, float softcap, const float* sinks, const void* gate, int gate_stride, int keep,
                                    int* err, cudaStream_t st) {
     return attn_simple_launch<__nv_bfloat16>(q, q_stride, out, positions, tok_seq, table, max_blocks, kpool, vpool, N,
                                              H, KV, HD, page, num_pages, window, scale, err, st, HDV, k_row, v_row, softcap,
-                                             sinks, gate, gate_stride);
+                                             sinks, gate, gate_stride, keep);
 }

@@ -305,6 +305,23 @@ __global__ void xielu_kernel(const T* __restrict__ in, T* __restrict__ out, size
     }
 }
 
+// ------------------------------------------------------------------------------------------------ squared ReLU
+template <typename T, bool VEC>
+__global__ void relu2_kernel(const T* __restrict__ in, T* __restrict__ out, size_t total) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (VEC) {
+        if (i * 8 >= total) return;
+        float v[8];
+        load8(in + i * 8, v);
+#pragma unroll
+        for (int e = 0; e < 8; e++) { v[e] = fmaxf(v[e], 0.0f); v[e] *= v[e]; }
+        store8(out + i * 8, v);
+    } else if (i < total) {
+        const float v = fmaxf(mb_load(in + i), 0.0f);
+        mb_store(out + i, v * v);
+    }
+}
+
 // ------------------------------------------------------------------------------------------------ rotation + K/V write
 // qkv[n] = [q (H*HD) | k (KV*HD) | v (KV*HD)] (+ bias).  q is rotated in place; k is rotated and written to its page,
 // v is written to its page (when pools are given).  freqs[i] is the angle per position step of pair i (RD/2 values);
@@ -598,6 +615,23 @@ MB_API int mb_xielu_f32(const void* in, void* out, long long total, float ap, fl
 }
 MB_API int mb_xielu_bf16(const void* in, void* out, long long total, float ap, float an, cudaStream_t st) {
     return xielu_launch<__nv_bfloat16>(in, out, total, ap, an, st);
+}
+
+template <typename T>
+static int relu2_launch(const void* in, void* out, long long total, cudaStream_t st) {
+    if (total <= 0) return 0;
+    const bool vec = total % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
+    const long long items = vec ? total / 8 : total;
+    if (vec) relu2_kernel<T, true><<<(unsigned)((items + 255) / 256), 256, 0, st>>>((const T*)in, (T*)out, (size_t)total);
+    else relu2_kernel<T, false><<<(unsigned)((items + 255) / 256), 256, 0, st>>>((const T*)in, (T*)out, (size_t)total);
+    MB_LAUNCH_CHECK();
+    return 0;
+}
+MB_API int mb_relu2_f32(const void* in, void* out, long long total, cudaStream_t st) {
+    return relu2_launch<float>(in, out, total, st);
+}
+MB_API int mb_relu2_bf16(const void* in, void* out, long long total, cudaStream_t st) {
+    return relu2_launch<__nv_bfloat16>(in, out, total, st);
 }
 
 MB_PDL_SWITCH(mb_elementwise_set_pdl)

@@ -30,7 +30,8 @@
 
 // MODE 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out (N, M); 3: bf16 out (N, M) =
 // xIELU of the product (ap z^2 + z / 2 for z > 0, an (e^z - 1 - z) + z / 2 otherwise); 4: as 1 with the gate of routed
-// experts, g = min(gate, ap), u = clamp(up, -ap, ap), out = g sigmoid(an g) (u + shift).
+// experts, g = min(gate, ap), u = clamp(up, -ap, ap), out = g sigmoid(an g) (u + shift); 5: bf16 out (N, M) = the square
+// of the product's positive part.
 //
 // Grouped form (tile_expert given): W is a stack of matrices of `expert_rows` rows each, and every tile of 128 rows of
 // act belongs to one of them -- tile_expert[token tile] says which, -1: the tile holds no rows and is passed over by
@@ -157,6 +158,13 @@ __global__ void __launch_bounds__(192, 1) gemm_tc5_kernel(const __grid_constant_
                     }
                 } else {
                     tmem_ld_wait();
+                    if (MODE == 5) {
+#pragma unroll
+                        for (int i = 0; i < 32; i++) {
+                            const float z = fmaxf(__bfloat162float(__float2bfloat16_rn(__uint_as_float(r[i]))), 0.0f);
+                            r[i] = __float_as_uint(z * z);
+                        }
+                    }
                     if (MODE == 3) {
 #pragma unroll
                         for (int i = 0; i < 32; i++) {
@@ -254,6 +262,11 @@ MB_API int mb_gemm_tc5_swiglu_bf16(const void* act, const void* W, void* out, in
 MB_API int mb_gemm_tc5_xielu_bf16(const void* act, const void* W, void* out, int N, int M, int K, float ap, float an,
                                   int* err, cudaStream_t st) {
     return tc5_launch<3>(act, W, out, N, M, K, err, st, ap, an);
+}
+// out (N, M) = max(act W^T, 0)^2
+MB_API int mb_gemm_tc5_relu2_bf16(const void* act, const void* W, void* out, int N, int M, int K, int* err,
+                                  cudaStream_t st) {
+    return tc5_launch<5>(act, W, out, N, M, K, err, st);
 }
 MB_API int mb_gemm_tc5_f32out(const void* act, const void* W, void* out, int N, int M, int K, int* err, cudaStream_t st) {
     return tc5_launch<2>(act, W, out, N, M, K, err, st);

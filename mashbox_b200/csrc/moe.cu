@@ -3,7 +3,8 @@
 //   moe_select     router logits z (N, E) float32 -> per token its `top` experts and their weights.  score s = sigmoid(z);
 //                  the choice is made on c = s + correction; the experts form `groups` equal runs of neighbours, a group
 //                  is worth the sum of its two largest c, and only experts of the `keep` best groups can be chosen;
-//                  the weight of a chosen expert is its s (not renormalised).  Ties go to the lower index.
+//                  the weight of a chosen expert is its s (not renormalised).  Ties go to the lower index.  Other kinds of
+//                  score: softmax(z); or z itself, with the softmax over the chosen ones as their weights
 //   moe_experts    for every (token, chosen expert): g = min(Wg h, L), u = clamp(Wu h, -L, L),
 //                  y = Wd (g sigmoid(alpha g) (u + 1)), left in float32 per (token, place)
 //   moe_combine    out[n] = sum over the places, in order, of weight * y
@@ -31,25 +32,34 @@ __device__ __forceinline__ int warp_argmax(const float* vals, int n, int lane) {
     return at;
 }
 
-// one warp per token; dynamic shared: s[E], c[E], gs[groups], kept[groups]
-// softmax: the scores are softmax(z) over all experts instead of sigmoid(z); worth_max: a group is worth its largest c
+// one warp per token; dynamic shared: s[E], c[E], gs[groups], kept[groups], won[top]
+// score 0: sigmoid(z); 1: softmax(z) over all experts; 2: z itself, the weights then being the softmax over the chosen
+// scores; bias (or null) is added to z first; worth_max: a group is worth its largest c
 // instead of the sum of its two largest; scale multiplies the weights; a row of z is z_stride floats long
-__global__ void moe_select_kernel(const float* __restrict__ z, int z_stride, const float* __restrict__ correction,
-                                  int* __restrict__ ids, float* __restrict__ wts, int E, int top, int groups, int keep,
-                                  int softmax, int worth_max, float scale) {
+__global__ void moe_select_kernel(const float* __restrict__ z, int z_stride, const float* __restrict__ bias,
+                                  const float* __restrict__ correction, int* __restrict__ ids, float* __restrict__ wts,
+                                  int E, int top, int groups, int keep, int score, int worth_max, float scale) {
     extern __shared__ float sm[];
     float* s = sm;
     float* c = sm + E;
     float* gs = sm + 2 * E;
     float* kept = gs + groups;
+    float* won = kept + groups;
     const int n = blockIdx.x, lane = threadIdx.x;
     const float* zr = z + (size_t)n * z_stride;
-    if (softmax) {
+    auto logit = [&](int e) { return bias ? zr[e] + bias[e] : zr[e]; };
+    if (score == 2) {
+        for (int e = lane; e < E; e += 32) {
+            const float v = logit(e);
+            s[e] = v;
+            c[e] = v + (correction ? correction[e] : 0.0f);
+        }
+    } else if (score == 1) {
         float m = -INFINITY;
-        for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e]);
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, logit(e));
         m = mb_warp_max(m);
         float sum = 0.0f;
-        for (int e = lane; e < E; e += 32) { const float v = expf(zr[e] - m); s[e] = v; sum += v; }
+        for (int e = lane; e < E; e += 32) { const float v = expf(logit(e) - m); s[e] = v; sum += v; }
         sum = mb_warp_sum(sum);
         for (int e = lane; e < E; e += 32) {
             const float v = s[e] / sum;
@@ -58,7 +68,7 @@ __global__ void moe_select_kernel(const float* __restrict__ z, int z_stride, con
         }
     } else {
         for (int e = lane; e < E; e += 32) {
-            const float v = 1.0f / (1.0f + expf(-zr[e]));
+            const float v = 1.0f / (1.0f + expf(-logit(e)));
             s[e] = v;
             c[e] = v + (correction ? correction[e] : 0.0f);
         }
@@ -91,11 +101,20 @@ __global__ void moe_select_kernel(const float* __restrict__ z, int z_stride, con
         __syncwarp();
         if (lane == 0) {
             ids[(size_t)n * top + kk] = at;
-            wts[(size_t)n * top + kk] = s[at] * scale;
+            won[kk] = s[at];
             c[at] = -INFINITY;
         }
         __syncwarp();
     }
+    float m = -INFINITY, sum = 0.0f;
+    if (score == 2) {
+        for (int kk = lane; kk < top; kk += 32) m = fmaxf(m, won[kk]);
+        m = mb_warp_max(m);
+        for (int kk = lane; kk < top; kk += 32) sum += expf(won[kk] - m);
+        sum = mb_warp_sum(sum);
+    }
+    for (int kk = lane; kk < top; kk += 32)
+        wts[(size_t)n * top + kk] = (score == 2 ? expf(won[kk] - m) / sum : won[kk]) * scale;
 }
 
 // sum over k of w[k] x[k], lanes side by side, x in shared memory (float); 16-byte loads of bf16 rows that allow them
@@ -195,13 +214,15 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
     mb_store(out + i, acc);
 }
 
-MB_API int mb_moe_select(const float* z, int z_stride, const float* correction, int* ids, float* wts, int N, int E, int top,
-                         int groups, int keep, int softmax, int worth_max, float scale, cudaStream_t st) {
+MB_API int mb_moe_select(const float* z, int z_stride, const float* bias, const float* correction, int* ids, float* wts, int N,
+                         int E, int top, int groups, int keep, int score, int worth_max, float scale, cudaStream_t st) {
     if (N == 0) return 0;
     if (E < 1 || top < 1 || top > E || groups < 1 || E % groups || keep < 1 || keep > groups || E > 8192 || z_stride < E) return -2;
     if ((long long)keep * (E / groups) < top) return -2;
-    moe_select_kernel<<<N, 32, (size_t)(2 * E + 2 * groups) * sizeof(float), st>>>(z, z_stride, correction, ids, wts, E, top,
-                                                                                   groups, keep, softmax, worth_max, scale);
+    const size_t smem = (size_t)(2 * E + 2 * groups + top) * sizeof(float);
+    if (score < 0 || score > 2 || smem > 48 * 1024) return -2;
+    moe_select_kernel<<<N, 32, smem, st>>>(z, z_stride, bias, correction, ids, wts, E, top, groups, keep, score, worth_max,
+                                           scale);
     MB_LAUNCH_CHECK();
     return 0;
 }

@@ -12,6 +12,7 @@
 //   retention_prep   from the product's rows [q | k | v | ...] in the storage type: the first R dims of every head of q
 //                    and k turn by position * freq_i (dim i with dim i + R/2), k times a constant after that; q, k, v
 //                    left in float32
+//   silu_rows        the same without rotation or constant, every value z as z / (1 + e^-z)
 //   retention_scan   the recurrence, token by token (decode steps, short portions, the whole float32 path)
 //   the split form   the same recurrence for long stretches.  The decay is a constant of the head, so a sequence can be
 //                    cut into segments that run side by side: every segment is scanned from a zero state (the first one
@@ -54,6 +55,34 @@ __global__ void retention_prep_kernel(const T* __restrict__ rows, int stride, in
     }
     const T* vs = row + v_off + (size_t)h * vdim;
     for (int c = threadIdx.x; c < vdim; c += blockDim.x) v[((size_t)n * H + h) * vdim + c] = mb_load(vs + c);
+}
+
+// out[n, c] = silu(rows[n, off + c]) in float32 for three neighbouring stretches of a row (q, k and v of C1, C1 and C2
+// values, one after the other from column 0).  grid (N, blocks over the row), VEC values a thread.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) silu_rows_kernel(const T* __restrict__ rows, int stride, float* __restrict__ q,
+                                                        float* __restrict__ k, float* __restrict__ v, int C1, int C2) {
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    if (c >= 2 * C1 + C2) return;
+    const size_t n = blockIdx.x;
+    const T* src = rows + n * stride + c;
+    float x[VEC];
+    if (VEC == 4 && sizeof(T) == 2) {
+        const uint2 w = *reinterpret_cast<const uint2*>(src);
+        x[0] = __uint_as_float(w.x << 16); x[VEC > 1 ? 1 : 0] = __uint_as_float(w.x & 0xffff0000u);
+        x[VEC > 2 ? 2 : 0] = __uint_as_float(w.y << 16); x[VEC > 3 ? 3 : 0] = __uint_as_float(w.y & 0xffff0000u);
+    } else {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) x[e] = mb_load(src + e);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; e++) x[e] = x[e] / (1.0f + expf(-x[e]));
+    float* dst = c < C1 ? q + n * C1 + c : c < 2 * C1 ? k + n * C1 + (c - C1) : v + n * C2 + (c - 2 * C1);
+    if (VEC == 4) {
+        *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[VEC > 1 ? 1 : 0], x[VEC > 2 ? 2 : 0], x[VEC > 3 ? 3 : 0]);
+    } else {
+        dst[0] = x[0];
+    }
 }
 
 // two floats in one 64-bit register pair, and the fused multiply-add on such pairs (one issue slot, two results, each
@@ -321,6 +350,29 @@ MB_API int mb_retention_prep_bf16(const void* rows, int stride, int q_off, int k
                                   float k_scale, cudaStream_t st) {
     return retention_prep_launch<bf16>((const bf16*)rows, stride, q_off, k_off, v_off, positions, freqs, q, k, v, N, H, dim,
                                        vdim, R, k_scale, st);
+}
+
+// rows (N, stride) = [q (C1) | k (C1) | v (C2) | ..]
+template <typename T>
+static int silu_rows_launch(const T* rows, int stride, float* q, float* k, float* v, int N, int C1, int C2, cudaStream_t st) {
+    if (N == 0) return 0;
+    if (C1 < 1 || C2 < 1 || stride < 2 * C1 + C2) return -2;
+    const bool vec = C1 % 4 == 0 && C2 % 4 == 0 && stride % 4 == 0 && ((uintptr_t)rows & 15) == 0 &&
+                     (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15) == 0;
+    const int items = (2 * C1 + C2) / (vec ? 4 : 1), blocks = (items + 255) / 256;
+    if (blocks > 65535) return -2;
+    if (vec) silu_rows_kernel<T, 4><<<dim3(N, blocks), 256, 0, st>>>(rows, stride, q, k, v, C1, C2);
+    else silu_rows_kernel<T, 1><<<dim3(N, blocks), 256, 0, st>>>(rows, stride, q, k, v, C1, C2);
+    MB_LAUNCH_CHECK();
+    return 0;
+}
+MB_API int mb_silu_rows_f32(const void* rows, int stride, float* q, float* k, float* v, int N, int C1, int C2,
+                            cudaStream_t st) {
+    return silu_rows_launch<float>((const float*)rows, stride, q, k, v, N, C1, C2, st);
+}
+MB_API int mb_silu_rows_bf16(const void* rows, int stride, float* q, float* k, float* v, int N, int C1, int C2,
+                             cudaStream_t st) {
+    return silu_rows_launch<bf16>((const bf16*)rows, stride, q, k, v, N, C1, C2, st);
 }
 
 static size_t rt_smem(int R4) {

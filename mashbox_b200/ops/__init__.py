@@ -202,6 +202,13 @@ def xielu(z, out, ap, an):
 
 
 # ------------------------------------------------------------------------------------------------ short convolutions
+def relu2(z, out):
+    """out = max(z, 0)^2, element by element"""
+    _cuda(z, out)
+    f = _fn("elementwise", "mb_relu2_" + _suffix(z.dtype), [c_void_p, c_void_p, c_ll, c_void_p])
+    _check(f(_p(z), _p(out), z.numel(), _stream()), "relu2")
+
+
 def short_conv(x, w, state, seq, out, residual=False):
     """out = (x if residual) + causal_conv(x): x, out (N, C) in the activation dtype, w (taps, C) float32, one filter per
     channel, held tap by tap (the transpose of how checkpoints store them).  state (slots, taps - 1, C) float32 (a view: rows C apart, slots state.stride(0) apart) holds every
@@ -494,6 +501,15 @@ def retention_prep(rows, q_off, k_off, v_off, positions, freqs, q, k, v, H, dim,
              rows.shape[0], H, dim, vdim, int(rotary_dim), float(k_scale), _stream()), "retention_prep")
 
 
+def silu_rows(rows, q, k, v):
+    """rows (N, C) of the activation dtype = [q | k | v | ..] -> q, k, v float32, every value z as silu(z)"""
+    _cuda(rows, q, k, v)
+    if k.shape != q.shape:
+        raise KernelError("silu_rows: queries and keys differ in width")
+    f = _fn("retention", "mb_silu_rows_" + _suffix(rows.dtype), [c_void_p, c_int] + [c_void_p] * 3 + [c_int] * 3 + [c_void_p])
+    _check(f(_p(rows), rows.stride(0), _p(q), _p(k), _p(v), rows.shape[0], q.shape[1], v.shape[1], _stream()), "silu_rows")
+
+
 # Steps with more than `chunk_tokens` tokens a sequence run the split form of the recurrence, in segments of
 # `segment_tokens` -- when the scan would leave the device short of blocks (fewer than `scan_blocks`): the split form walks
 # every token twice, which pays only while the scan's blocks do not fill the multiprocessors.
@@ -640,19 +656,24 @@ def sigmoid_attention_tc5(q, out, items, n_items, q_start, q_len, pos0, seq_row,
 
 
 # ------------------------------------------------------------------------------------------------ routed experts
-def moe_select(z, correction, ids, wts, groups=1, keep=1, experts=None, softmax=False, worth="top2", scale=1.0):
-    """z (N, >= E) float32 router logits (E = experts, default: every column) -> ids (N, top) int32, wts (N, top) float32:
-    scores sigmoid(z), or softmax(z) over the E experts; chosen by score + correction among the experts of the `keep` best
+MOE_SCORES = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
+
+
+def moe_select(z, correction, ids, wts, groups=1, keep=1, experts=None, score="sigmoid", worth="top2", scale=1.0, bias=None):
+    """z (N, >= E) float32 router logits (E = experts, default: every column), bias (E,) float32 added to them (None: none)
+    -> ids (N, top) int32, wts (N, top) float32: scores sigmoid(z), softmax(z) over the E experts, or z itself with the
+    softmax over the chosen ones as their weights ("softmax_chosen"); chosen by score + correction among the experts of the `keep` best
     of `groups` runs of neighbours (a run's worth: the sum of its two largest, "top2", or its largest, "max"); the
     weights are the chosen experts' scores times `scale`"""
-    _cuda(z, correction, ids, wts)
+    _cuda(z, bias, correction, ids, wts)
     N = z.shape[0]
     E = int(experts) if experts is not None else z.shape[1]
-    if worth not in ("top2", "max"):
-        raise KernelError(f"moe_select: a group's worth is top2 or max, not {worth!r}")
-    f = _fn("moe", "mb_moe_select", [c_void_p, c_int] + [c_void_p] * 3 + [c_int] * 7 + [c_float, c_void_p])
-    _check(f(_p(z), z.stride(0), _p(correction), _p(ids), _p(wts), N, E, ids.shape[1], int(groups), int(keep),
-             int(bool(softmax)), int(worth == "max"), float(scale), _stream()), "moe_select")
+    if worth not in ("top2", "max") or score not in MOE_SCORES:
+        raise KernelError(f"moe_select: a group's worth is top2 or max, not {worth!r}; a score one of "
+                          f"{', '.join(MOE_SCORES)}, not {score!r}")
+    f = _fn("moe", "mb_moe_select", [c_void_p, c_int] + [c_void_p] * 4 + [c_int] * 7 + [c_float, c_void_p])
+    _check(f(_p(z), z.stride(0), _p(bias), _p(correction), _p(ids), _p(wts), N, E, ids.shape[1], int(groups), int(keep),
+             MOE_SCORES[score], int(worth == "max"), float(scale), _stream()), "moe_select")
 
 
 def _expert_views(wg, wu, wd):
@@ -1050,6 +1071,23 @@ def linear_xielu(a, w, out, ap, an):
                                                    c_void_p, c_void_p])
     _check(f(_p(a), _p(w), _p(out), N, out.shape[1], K, float(ap), float(an), _p(error_word(a.device)), _stream()),
            "gemm_tc5_xielu")
+    return out
+
+
+def fused_relu2_supports(N, F, K, dtype):
+    """the up product of a bfloat16 prompt portion with the squared ReLU in its epilogue (the tcgen05 product)"""
+    return dtype == torch.bfloat16 and tc5_supports(N, F, K, "swiglu")
+
+
+def linear_relu2(a, w, out):
+    """a (N, K) bf16, w (F, K) bf16 -> out (N, F) bf16 = max(a W^T, 0)^2, one kernel; shapes fused_relu2_supports() takes"""
+    _cuda(a, w, out)
+    N, K = a.shape
+    if not (fused_relu2_supports(N, out.shape[1], K, a.dtype) and a.is_contiguous() and w.is_contiguous()
+            and out.is_contiguous()):
+        raise KernelError("linear_relu2: no fused kernel takes these sizes")
+    f = _fn("gemm_tc5", "mb_gemm_tc5_relu2_bf16", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(f(_p(a), _p(w), _p(out), N, out.shape[1], K, _p(error_word(a.device)), _stream()), "gemm_tc5_relu2")
     return out
 
 
@@ -1509,18 +1547,21 @@ def gated_scan(q, k, v, g, o, state, seq, H, G, dim, vdim, per_head):
 
 # ------------------------------------------------------------------------------------------------ normed, rotated heads
 def norm_rope_kv_write(rows, qw, kw, eps, freqs, RD, pairing, gain, positions, tok_row, table, kpool, vpool, H, KV, DK,
-                       DV, page, num_pages, err):
-    """rows (N, >= (H + KV) DK + KV DV) = [q | k | v | ..]: every q and k head divided by its root mean square and
-    multiplied by qw / kw (DK values; None: no norm), its first RD values rotated by the token's position (freqs (RD/2,)
-    float32 or None; pairing 0 adjacent, 1 halves; cos and sin times gain); q back in place, k and v into the pages:
-    kpool (pages, KV, page, DK), vpool (pages, KV, page, DV); both None: q only"""
-    _cuda(rows, qw, kw, freqs, positions, tok_row, table, kpool, vpool)
+                       DV, page, num_pages, err, norm="before", v_keep=None, v_first=None, lam=0.0):
+    """rows (N, >= (H + KV) DK + KV DV) = [q | k | v | ..]: the first RD values of every q and k head rotated by the token's
+    position (freqs (RD/2,) float32 or None; pairing 0 adjacent, 1 halves; cos and sin times gain), the head divided by its
+    root mean square and multiplied by qw / kw (DK values; None: no weights) before or after that (norm: "before" |
+    "after" | None); q back in place, k and v into the pages: kpool (pages, KV, page, DK), vpool (pages, KV, page, DV); both
+    None: q only.  v_keep (N, KV DV): receives the values as they are; v_first (N, KV DV): what is cached is
+    (1 - lam) v + lam v_first."""
+    _cuda(rows, qw, kw, freqs, positions, tok_row, table, kpool, vpool, v_keep, v_first)
     f = _fn("rotary_rows", "mb_norm_rope_kv_write_" + _suffix(rows.dtype),
-            [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
-             c_int, c_void_p, c_void_p] + [c_int] * 7 + [c_void_p, c_void_p])
-    _check(f(_p(rows), rows.stride(0), _p(qw), _p(kw), float(eps), _p(freqs), int(RD), int(pairing), float(gain),
-             _p(positions), _p(tok_row), _p(table), table.shape[1], _p(kpool), _p(vpool), rows.shape[0], H, KV, DK, DV, page,
-             num_pages, _p(err), _stream()), "norm_rope_kv_write")
+            [c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
+             c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float] + [c_int] * 7 + [c_void_p, c_void_p])
+    _check(f(_p(rows), rows.stride(0), _p(qw), _p(kw), float(eps), {None: 0, "before": 1, "after": 2}[norm], _p(freqs),
+             int(RD), int(pairing), float(gain), _p(positions), _p(tok_row), _p(table), table.shape[1], _p(kpool), _p(vpool),
+             _p(v_keep), _p(v_first), float(lam), rows.shape[0], H, KV, DK, DV, page, num_pages, _p(err), _stream()),
+           "norm_rope_kv_write")
 
 
 def latent_rope(q, q_head, q_off, qa, qa_head, qa_off, rows, kr_off, pool, pool_off, freqs, RD, W, pairing, gain,
@@ -1540,19 +1581,20 @@ def latent_rope(q, q_head, q_off, qa, qa_head, qa_off, rows, kr_off, pool, pool_
 
 
 def attention_general(q, q_stride, out, positions, tok_seq, table, kpool, vpool, H, KV, DK, DV, page, num_pages, window,
-                      scale, err, softcap=None, sinks=None, gate=None):
+                      scale, err, softcap=None, sinks=None, gate=None, keep=0):
     """The plain paged attention kernel in its general form: keys of DK and values of DV values (the pools' rows may be
     wider: their last dimension is the distance between two positions), scores capped by softcap tanh(s / softcap), a
-    sink per query head in the denominator (sinks (H,) float32), the result of head h times sigmoid(gate[n, h])"""
+    sink per query head in the denominator (sinks (H,) float32), the result of head h times sigmoid(gate[n, h]); the first
+    `keep` positions stay visible behind the window"""
     _cuda(q, out, positions, tok_seq, table, kpool, vpool, sinks, gate)
     N = out.shape[0]
     f = _fn("attention_simple", "mb_attn_simple_ext_" + _suffix(out.dtype),
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 10
-            + [c_float, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
+            + [c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p])
     _check(f(_p(q), q_stride, _p(out), _p(positions), _p(tok_seq), _p(table), table.shape[1], _p(kpool), _p(vpool), N, H,
              KV, DK, DV, kpool.shape[-1], vpool.shape[-1], page, num_pages, window or 0, float(scale),
-             float(softcap or 0.0), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, _p(err), _stream()),
-           "attention_general")
+             float(softcap or 0.0), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, int(keep), _p(err),
+             _stream()), "attention_general")
 
 
 def attention_general_mma_supports(DK, DV):
@@ -1567,7 +1609,7 @@ def _general_mma_library(DK, DV):
 
 def attention_general_mma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_start, q_len, pos0, part_base, seq_row,
                           table, part_o, part_ml, max_splits, H, KV, DK, DV, page, num_pages, window, scale, err,
-                          softcap=None, sinks=None, gate=None):
+                          softcap=None, sinks=None, gate=None, keep=0):
     """attention_general on tensor cores (bfloat16): items are (sequence, row tile, split, splits) quadruples of the
     prompt form (tiles of 64 packed rows) or, with decode, of the decode form (at most 16); split items leave partial
     sums in part_o / part_ml for attention_general_merge.  Compiled for the pair (DK, DV) the first time it is asked for."""
@@ -1576,12 +1618,13 @@ def attention_general_mma(q, q_stride, out, kpool, vpool, items, n_items, decode
         raise KernelError(f"attention_general_mma: no kernel for {out.dtype} with widths {DK} and {DV}")
     f = _fn(_general_mma_library(DK, DV), "mb_attn_general_bf16",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int] + [c_void_p] * 6 + [c_int]
-            + [c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
+            + [c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p,
+                                                            c_void_p])
     _check(f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), kpool.shape[-1], vpool.shape[-1], _p(items), int(n_items),
              1 if decode else 0, _p(q_start), _p(q_len), _p(pos0), _p(part_base), _p(seq_row), _p(table), table.shape[1],
              _p(part_o), _p(part_ml), max_splits, H, KV, DK, DV, page, num_pages, window or 0, float(scale),
-             float(softcap or 0.0), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, _p(err), _stream()),
-           "attention_general_mma")
+             float(softcap or 0.0), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, int(keep), _p(err),
+             _stream()), "attention_general_mma")
 
 
 def attention_general_merge(part_o, part_ml, part_tok, n_part, out, H, DK, DV, max_splits, sinks=None, gate=None):

@@ -53,11 +53,12 @@ class PagedAttention:
     once, say) hands its pools in."""
 
     def __init__(self, heads, kv_heads, head_dim, window=None, scale=None, vdim=None, softcap=None, sinks=False,
-                 gated=False):
+                 gated=False, keep_first=0):
         """vdim: the width of a value when it is not the key's (the result is heads * vdim wide); softcap: scores become
         softcap tanh(s / softcap); sinks: attend() is handed one number per query head that joins the softmax's
         denominator without a value; gated: attend() is handed a gate per token and query head (the head's result
-        times its sigmoid).  Any of the four, or pools whose rows are wider than what is read of them, make the
+        times its sigmoid); keep_first: behind the window the first `keep_first` positions stay visible.  Any of
+        the five, or pools whose rows are wider than what is read of them, make the
         attention *general*: it runs on the kernels that take all of that."""
         self.H, self.KV, self.HD = int(heads), int(kv_heads), int(head_dim)
         if self.H % self.KV:
@@ -66,7 +67,8 @@ class PagedAttention:
         self.scale = float(scale) if scale else self.HD ** -0.5
         self.VD = int(vdim) if vdim else self.HD
         self.softcap = float(softcap) if softcap else None
-        self.general = self.VD != self.HD or self.softcap is not None or bool(sinks) or bool(gated)
+        self.keep = int(keep_first) if self.window else 0       # without a window every position is visible anyway
+        self.general = self.VD != self.HD or self.softcap is not None or bool(sinks) or bool(gated) or self.keep > 0
 
     # ------------------------------------------------------------------------------------------ planning
     def uses_mma(self, ctx):
@@ -90,7 +92,7 @@ class PagedAttention:
 
     def plan_key(self):
         # everything the work list depends on: the head size decides the kernel and its rows per tile
-        return ("attention", self.H // self.KV, self.KV, self.HD, self.window, self.general)
+        return ("attention", self.H // self.KV, self.KV, self.HD, self.window, self.keep, self.general)
 
     def prepare(self, ctx):
         """Work list of the flash kernel for this step: (sequence, row tile, split, splits) per block, decode-form
@@ -120,7 +122,8 @@ class PagedAttention:
         def key_tiles(s):
             hi = ctx.pos0[s] + ctx.q_len[s]
             lo = max(0, ctx.pos0[s] - self.window + 1) if self.window else 0
-            return -(-(hi - lo // KEY_TILE * KEY_TILE) // KEY_TILE)
+            front = min(-(-self.keep // KEY_TILE), lo // KEY_TILE)          # tiles of kept positions before the window's
+            return front + -(-(hi - lo // KEY_TILE * KEY_TILE) // KEY_TILE)
 
         # Decode-form sequences on the TMA kernel: when they can all be cut into the same number of splits (set by the
         # longest of them; a shorter one leaves some of its splits empty) the blocks of a sequence and kv head are
@@ -260,14 +263,14 @@ class PagedAttention:
                                               ctx.dev("q_start"), ctx.dev("q_len"), ctx.dev("pos0"),
                                               ctx.dev(nm + "part_base"), ctx.dev("seq_row"), table, part_o, part_ml, ms, H,
                                               KV, self.HD, self.VD, page, pages, self.window, self.scale, ctx.err,
-                                              self.softcap, sinks, gate)
+                                              self.softcap, sinks, gate, keep=self.keep)
             if n_part:
                 ops.attention_general_merge(part_o, part_ml, ctx.dev(nm + "part_tok"), n_part, out, H, self.HD, self.VD, ms,
                                             sinks, gate)
             return
         ctx.ops.attention_general(q, width, out, ctx.dev("positions"), ctx.dev("tok_row"), table, kpool, vpool, self.H,
                                   self.KV, self.HD, self.VD, ctx.cache.page_size, ctx.cache.pool_pages, self.window,
-                                  self.scale, ctx.err, self.softcap, sinks, gate)
+                                  self.scale, ctx.err, self.softcap, sinks, gate, keep=self.keep)
 
 
 class Attention(PagedAttention):
@@ -378,8 +381,10 @@ register("mixer", "attention", Attention)
 
 class GatedAttention(PagedAttention):
     """Grouped-query attention whose keys and values may differ in width, with, each optional: an RMS norm of every q
-    and k head before the rotation (`qk_norm`: weights `<q>.norm` and `<k>.norm` of head_dim values, shared by the
-    heads), a rotation of the first dims of a head (`position`, any rope spec), capped scores (`softcap`), a sink in
+    and k head before the rotation (`qk_norm` True: weights `<q>.norm` and `<k>.norm` of head_dim values, shared by the
+    heads) or after it (`qk_norm` "after": no weights), a sliding window (`window`) behind which the first `keep_first`
+    positions stay visible, values mixed with those of another layer of the same step (`value_mix`: "keep" leaves this
+    layer's values for the others, "mix" caches (1 - lam) v + lam v_kept, lam stored as `<vmix>`), a rotation of the first dims of a head (`position`, any rope spec), capped scores (`softcap`), a sink in
     the softmax's denominator (`sink`: "unit" -- a sink of score zero, so one is added to the denominator -- or the name
     of a tensor with one number per query head, or None) and a gate per token and query head (`gate`: head h's result
     times sigmoid(Wg h)_h, Wg stored as `<g>`).  No biases.
@@ -392,12 +397,16 @@ class GatedAttention(PagedAttention):
     attention kernel takes cap, sink and gate in.  Norms, angles, scores and the softmax are float32."""
 
     def __init__(self, hidden, heads, kv_heads, head_dim, vdim=None, scale=None, softcap=None, qk_norm=False, eps=1e-6,
-                 sink=None, gate=False, position=None, window=None, prefix="", names=None):
+                 sink=None, gate=False, position=None, window=None, keep_first=0, value_mix=None, prefix="", names=None):
         super().__init__(heads, kv_heads, head_dim, window, scale, vdim=vdim, softcap=softcap, sinks=sink is not None,
-                         gated=gate)
+                         gated=gate, keep_first=keep_first)
         self.general = True         # this mixer's own path: separate key and value pools, q/k norms
-        self.D, self.eps, self.qk_norm, self.sink, self.gate = int(hidden), float(eps), bool(qk_norm), sink, bool(gate)
-        n = dict(q="q", k="k", v="v", g="g", o="o", q_norm="q.norm", k_norm="k.norm")
+        self.D, self.eps, self.sink, self.gate = int(hidden), float(eps), sink, bool(gate)
+        if qk_norm not in (True, False, None, "after") or value_mix not in (None, "keep", "mix"):
+            raise ConfigError(f"this attention has no q/k norm {qk_norm!r} or value mixing {value_mix!r}")
+        self.norm_at = "after" if qk_norm == "after" else ("before" if qk_norm else None)
+        self.value_mix, self.lam = value_mix, 0.0
+        n = dict(q="q", k="k", v="v", g="g", o="o", q_norm="q.norm", k_norm="k.norm", vmix="vmix")
         n.update(names or {})
         self.n = {k: prefix + v for k, v in n.items()}
         self.sink_name = prefix + sink if sink not in (None, "unit") else None
@@ -412,7 +421,9 @@ class GatedAttention(PagedAttention):
         H, KV, HD, VD, D = self.H, self.KV, self.HD, self.VD, self.D
         out = [Want(self.n["q"], (H * HD, D), "matrix"), Want(self.n["k"], (KV * HD, D), "matrix"),
                Want(self.n["v"], (KV * VD, D), "matrix"), Want(self.n["o"], (D, H * VD), "matrix")]
-        if self.qk_norm:
+        if self.value_mix == "mix":
+            out.append(Want(self.n["vmix"], (), "vector"))
+        if self.norm_at == "before":
             out += [Want(self.n["q_norm"], (HD,), "vector"), Want(self.n["k_norm"], (HD,), "vector")]
         if self.gate:
             out.append(Want(self.n["g"], (H, D), "matrix"))
@@ -429,7 +440,9 @@ class GatedAttention(PagedAttention):
             parts.append(torch.zeros((8 - rows % 8, self.D), dtype=parts[0].dtype, device=parts[0].device))
         self.w_in = torch.cat(parts, 0).contiguous()
         self.wo = t("o")
-        self.qw, self.kw = (t("q_norm"), t("k_norm")) if self.qk_norm else (None, None)
+        self.qw, self.kw = (t("q_norm"), t("k_norm")) if self.norm_at == "before" else (None, None)
+        if self.value_mix == "mix":
+            self.lam = float(t("vmix").float().cpu())
         if self.sink == "unit":
             self.sinks = torch.zeros(self.H, dtype=torch.float32, device=env.device)
         elif self.sink_name:
@@ -440,7 +453,8 @@ class GatedAttention(PagedAttention):
                 raise ConfigError("this attention rotates in its own kernel; its position part must hand it frequencies")
 
     def cache_need(self):
-        return CacheNeed("window" if self.window else "full", ((self.KV, self.HD), (self.KV, self.VD)), self.window)
+        return CacheNeed("window" if self.window else "full", ((self.KV, self.HD), (self.KV, self.VD)), self.window,
+                         self.keep)
 
     def state_need(self):
         return None
@@ -456,9 +470,13 @@ class GatedAttention(PagedAttention):
         if self.position is not None:
             freqs, rd, pairing = self.position.rotation()
             gain = getattr(self.position, "gain", 1.0)
+        # the layer whose values others mix in runs first in the step and leaves them in a buffer of the step's tokens
+        kept = ctx.ws.get("values_kept", N, (KV * VD,), ctx.dtype) if self.value_mix else None
         ops.norm_rope_kv_write(rows, self.qw, self.kw, self.eps, freqs, rd, pairing, gain, ctx.dev("positions"),
                                ctx.dev("tok_row"), table, kpool if run.write else None, vpool if run.write else None, H, KV,
-                               HD, VD, page, pages, ctx.err)
+                               HD, VD, page, pages, ctx.err, norm=self.norm_at,
+                               v_keep=kept if self.value_mix == "keep" else None,
+                               v_first=kept if self.value_mix == "mix" else None, lam=self.lam)
         o = ctx.ws.get("gattn_out", N, (H * VD,), ctx.dtype)
         off = (H + KV) * HD + KV * VD
         gate = rows[:, off:off + H] if self.gate else None

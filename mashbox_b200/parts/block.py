@@ -133,22 +133,26 @@ register("block", "prenorm_depth", DepthAveragedBlock)
 
 
 class ParallelBlock:
-    """x += mixer(conv(norm1(x))) + ffn(norm2(x)): both sublayers read the same stream, each through a norm of its own.
+    """x += mixer(conv(norm1(x))) + ffn(norm2(x)): both sublayers read the same stream, each through a norm of its own,
+    or (`one_norm`) both through norm1.
 
     `mixer_conv` (optional): a short causal convolution on what the mixer reads.  `ffn` may be None.  The two outputs
     stay pending (delta of the mixer, None, delta of the feed-forward) and the next norm kernel adds both into the
-    float32 stream; when the two norms are of one kind, width and eps, one kernel makes both from one sum of squares.
+    float32 stream; when the two norms are of one kind, width and eps, one kernel makes both from one sum of squares
+    (with one norm there is one output, which both read).
     The layer's state (what its convolutions carry across steps) is one flat float32 tensor per request: the input
     convolution's stretch first, then the mixer's."""
 
-    def __init__(self, prefix, mixer, norm1, norm2=None, ffn=None, mixer_conv=None, names=None):
+    def __init__(self, prefix, mixer, norm1, norm2=None, ffn=None, mixer_conv=None, names=None, one_norm=False):
         n = dict(norm1="norm1", norm2="norm2", conv="canon1")
         n.update(names or {})
         self.norm1 = make("norm", norm1, name=prefix + n["norm1"])
         self.conv = make("conv", mixer_conv, name=prefix + n["conv"]) if mixer_conv is not None else None
         self.mixer = make("mixer", mixer, prefix=prefix)
         self.ffn = make("feed_forward", ffn, prefix=prefix) if ffn is not None else None
-        self.norm2 = make("norm", norm2 or norm1, name=prefix + n["norm2"]) if self.ffn is not None else None
+        self.norm2 = None
+        if self.ffn is not None and not one_norm:
+            self.norm2 = make("norm", norm2 or norm1, name=prefix + n["norm2"])
         off = 0
         for part in (self.conv, self.mixer):
             if part is not None and hasattr(part, "state_floats"):
@@ -182,7 +186,7 @@ class ParallelBlock:
     def forward(self, ctx, x, pending, run):
         ctx.after_norm = None
         conv_done = False
-        if self.ffn is not None and hasattr(self.norm1, "forward_pair") and type(self.norm2) is type(self.norm1) \
+        if self.norm2 is not None and hasattr(self.norm1, "forward_pair") and type(self.norm2) is type(self.norm1) \
                 and (self.norm1.width, self.norm1.eps) == (self.norm2.width, self.norm2.eps):
             # a step in which every sequence brings one token (N == S follows from the lengths of the step's arrays): the
             # input convolution is the same kernel's work
@@ -194,7 +198,7 @@ class ParallelBlock:
                 conv_done = True
         else:
             a = self.norm1.forward(ctx, x, pending)
-            b = self.norm2.forward(ctx, x, None) if self.ffn is not None else None
+            b = self.norm2.forward(ctx, x, None) if self.norm2 is not None else a
         if self.conv is not None and not conv_done:
             a = self.conv.forward(ctx, a, run.state_id)
         delta, bias = self.mixer.forward(ctx, a, run)

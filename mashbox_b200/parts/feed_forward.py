@@ -57,6 +57,41 @@ def _softplus(t):
     return max(t, 0.0) + math.log1p(math.exp(-abs(t)))
 
 
+class DenseReluSquared:
+    """relu(h Wu^T)^2 Wd^T, no biases; the square is float32 arithmetic on the product's outputs."""
+    graph_safe = True       # forward() depends on the batch only through the lengths of the step's arrays
+
+    def __init__(self, hidden, intermediate, prefix="", names=None):
+        self.D, self.F = int(hidden), int(intermediate)
+        n = dict(up="ffn_up.weight", down="ffn_down.weight")
+        n.update(names or {})
+        self.names = {k: prefix + v for k, v in n.items()}
+        self.wu = self.wd = None
+
+    def wants(self):
+        return [Want(self.names["up"], (self.F, self.D), "matrix"), Want(self.names["down"], (self.D, self.F), "matrix")]
+
+    def bind(self, tensors, env):
+        self.wu, self.wd = tensors[self.names["up"]], tensors[self.names["down"]]
+
+    def forward(self, ctx, h, out="delta"):
+        """out: the workspace buffer the result is left in"""
+        N = ctx.N
+        a = ctx.ws.get("ffn_act", N, (self.F,), ctx.dtype)
+        if ctx.ops.fused_relu2_supports(N, self.F, self.D, ctx.dtype) and h.is_contiguous():
+            ctx.ops.linear_relu2(h, self.wu, a)             # the product with the activation in its epilogue
+        else:
+            z = ctx.ws.get("ffn_up", N, (self.F,), ctx.dtype)
+            ctx.ops.linear(h, self.wu, out=z)
+            ctx.ops.relu2(z, a)
+        y = ctx.ws.get(out, N, (self.D,), ctx.dtype)
+        ctx.ops.linear(a, self.wd, out=y)
+        return y, None
+
+
+register("feed_forward", "dense_relu2", DenseReluSquared)
+
+
 class DenseXielu:
     """act(h Wu^T) Wd^T with the xIELU activation: act(z) = ap z^2 + z/2 for z > 0 and an (e^z - 1 - z) + z/2 otherwise,
     ap = softplus(p), an = 1/2 + softplus(q); the layer's two numbers (p, q) are one stored tensor.  The activation is

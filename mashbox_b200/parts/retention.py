@@ -1,4 +1,5 @@
-"""The retention mixer: linear attention with one fixed decay per head, no softmax and no denominator.
+"""The retention mixer: linear attention with one fixed decay per head, no softmax and no denominator (and, at the end of
+the file, lightning attention, which is the same recurrence between other ends).
 
     q = Wq h, k = Wk h   (heads x dim);   v = Wv h   (heads x vdim);   no biases
     the first R dims of every head of q and k are rotated by position * f_i (a `rope` position part: halves pairing,
@@ -68,6 +69,19 @@ class Retention:
     def prepare(self, ctx):
         pass
 
+    def prepare_rows(self, ctx, rows, q, k, v):
+        """q, k, v in float32 from the rows of the product"""
+        H, dim = self.H, self.dim
+        freqs, rd = (None, 0)
+        if self.position is not None:
+            freqs, rd, _ = self.position.rotation()
+        ctx.ops.retention_prep(rows, 0, H * dim, 2 * H * dim, ctx.dev("positions"), freqs, q, k, v, H, dim, self.vdim, rd,
+                               dim ** -0.5)
+
+    def gated(self, ctx, o, gate, a):
+        """a = the recurrence's output, normed and gated"""
+        ctx.ops.gated_rms(o, gate, None, a, self.H, self.vdim, self.eps, silu=True)
+
     def forward(self, ctx, h, run, out="delta"):
         import torch
         ops, N = ctx.ops, ctx.N
@@ -78,11 +92,7 @@ class Retention:
         q = ctx.ws.get("retention_q", N, (H * dim,), f32)
         k = ctx.ws.get("retention_k", N, (H * dim,), f32)
         v = ctx.ws.get("retention_v", N, (H * vdim,), f32)
-        freqs, rd = (None, 0)
-        if self.position is not None:
-            freqs, rd, _ = self.position.rotation()
-        ops.retention_prep(rows, 0, H * dim, 2 * H * dim, ctx.dev("positions"), freqs, q, k, v, H, dim, vdim, rd,
-                           dim ** -0.5)
+        self.prepare_rows(ctx, rows, q, k, v)
         o = ctx.ws.get("retention_o", N, (H * vdim,), f32)
         off = self.state_offset
         state = ctx.cache.state[run.state_id][:, off:off + self.state_floats()]
@@ -95,10 +105,40 @@ class Retention:
         ops.retention(q, k, v, self.decay, o, state, (ctx.dev("q_start"), ctx.dev("q_len"), ctx.dev("state_slot")), H, dim,
                       vdim, chunked=chunked, carry=carry)
         a = ctx.ws.get("retention_gated", N, (H * vdim,), ctx.dtype)
-        ops.gated_rms(o, rows[:, 2 * H * dim + H * vdim:], None, a, H, vdim, self.eps, silu=True)
+        self.gated(ctx, o, rows[:, 2 * H * dim + H * vdim:], a)
         y = ctx.ws.get(out, N, (self.D,), ctx.dtype)
         ops.linear(a, self.wo, out=y)
         return y, None
 
 
 register("mixer", "retention", Retention)
+
+
+class LightningAttention(Retention):
+    """Lightning attention: retention's recurrence on activated projections, one weighted norm over all heads at once.
+
+        q = silu(Wq h), k = silu(Wk h)   (heads x dim);   v = silu(Wv h)   (heads x vdim);   no rotation, no other scale
+        per head and token:  S <- decay_h S + k v^T;  o = S^T q
+        out = Wo (rms(concat_h o_h) n * sigmoid(Wg h))          n: heads x vdim values"""
+
+    def __init__(self, hidden, heads, dim, vdim, decay, eps, prefix="", names=None):
+        n = dict(q="q", k="k", v="v", g="g", o="o", norm="norm")
+        n.update(names or {})
+        super().__init__(hidden, heads, dim, vdim, decay, eps, None, prefix, n)
+        self.norm_w = None
+
+    def wants(self):
+        return super().wants() + [Want(self.n["norm"], (self.H * self.vdim,), "vector")]
+
+    def bind(self, tensors, env):
+        super().bind(tensors, env)
+        self.norm_w = tensors[self.n["norm"]]
+
+    def prepare_rows(self, ctx, rows, q, k, v):
+        ctx.ops.silu_rows(rows, q, k, v)
+
+    def gated(self, ctx, o, gate, a):
+        ctx.ops.gated_rms(o, gate, self.norm_w, a, 1, self.H * self.vdim, self.eps, silu=False)
+
+
+register("mixer", "lightning", LightningAttention)

@@ -5,7 +5,9 @@
     `keep` best runs cannot be chosen; the `top` largest c are chosen; out = sum over the chosen of s_e expert_e(h)
     expert: g = min(Wg h, limit);  u = clamp(Wu h, -limit, limit);  Wd (g sigmoid(alpha g) (u + 1))
 
-Variants, all constructor parameters: the scores may be softmax(z) over all experts (`score="softmax"`); a run may be
+Variants, all constructor parameters: the scores may be softmax(z) over all experts (`score="softmax"`), or the choice may
+be made on z itself and the weights be the softmax over the chosen z alone (`score="softmax_chosen"`); z may have a bias per
+expert (`router_bias`: its tensor), which counts in choice and weights alike; a run may be
 worth its largest c alone (`group_worth="max"`); the weights may be multiplied by a constant (`scale`); the expert may be
 the plain gated form Wd (silu(Wg h) * (Wu h)) (`limit=None, alpha=1, shift=0`: no clamps, nothing added to u); and an
 expert that every token uses (`shared`: the spec of a feed-forward part, its tensors under `shared_prefix`) may be added,
@@ -30,16 +32,17 @@ class RoutedExperts:
 
     def __init__(self, hidden, intermediate, experts, top, limit, groups=1, keep=1, alpha=1.702, correction=True,
                  score="sigmoid", group_worth="top2", scale=1.0, shift=1.0, shared=None, shared_prefix="mlp.shared.",
-                 shared_gate=None, prefix="", names=None):
+                 shared_gate=None, router_bias=None, prefix="", names=None):
         self.D, self.F, self.E, self.top = int(hidden), int(intermediate), int(experts), int(top)
         self.groups, self.keep = int(groups or 1), int(keep or 1)
         self.limit = float(limit) if limit is not None else float("inf")
         self.alpha, self.has_correction = float(alpha), bool(correction)
-        if score not in ("sigmoid", "softmax") or group_worth not in ("top2", "max"):
+        if score not in ("sigmoid", "softmax", "softmax_chosen") or group_worth not in ("top2", "max"):
             raise ConfigError(f"routed experts: score {score!r} / group worth {group_worth!r} are not known")
         self.score, self.group_worth, self.scale, self.shift = score, group_worth, float(scale), float(shift)
         self.shared = make("feed_forward", shared, prefix=prefix + shared_prefix) if shared is not None else None
         self.shared_gate = prefix + shared_gate if (shared_gate and self.shared is not None) else None
+        self.router_bias = prefix + router_bias if router_bias else None
         if self.E % self.groups or not 1 <= self.keep <= self.groups:
             raise ConfigError(f"{experts} experts do not form {groups} equal groups of which {keep} are kept")
         if not 1 <= self.top <= self.keep * (self.E // self.groups):
@@ -47,7 +50,7 @@ class RoutedExperts:
         n = dict(router="mlp.router", correction="mlp.correction", expert="mlp.e{}.", gate="gate", up="up", down="down")
         n.update(names or {})
         self.n = {k: (v if k in ("gate", "up", "down") else prefix + v) for k, v in n.items()}
-        self.wr = self.corr = self.wg = self.wu = self.wd = None
+        self.wr = self.br = self.corr = self.wg = self.wu = self.wd = None
 
     @property
     def graph_safe(self):
@@ -58,6 +61,8 @@ class RoutedExperts:
 
     def wants(self):
         out = [Want(self.n["router"], (self.E, self.D), "matrix")]
+        if self.router_bias:
+            out.append(Want(self.router_bias, (self.E,), "vector"))
         if self.has_correction:
             out.append(Want(self.n["correction"], (self.E,), "vector"))
         for e in range(self.E):
@@ -73,6 +78,7 @@ class RoutedExperts:
     def bind(self, tensors, env):
         import torch
         self.wr = tensors[self.n["router"]]
+        self.br = tensors[self.router_bias] if self.router_bias else None
         if self.shared is not None:
             self.shared.bind(tensors, env)
         if self.shared_gate:            # the gate's logit is one more row of the router's product
@@ -90,8 +96,8 @@ class RoutedExperts:
         ops.linear(h, self.wr, out=z, out_dtype=torch.float32)
         ids = ctx.ws.get("router_ids", N, (self.top,), torch.int32)
         wts = ctx.ws.get("router_weights", N, (self.top,), torch.float32)
-        ops.moe_select(z, self.corr, ids, wts, self.groups, self.keep, experts=self.E, softmax=self.score == "softmax",
-                       worth=self.group_worth, scale=self.scale)
+        ops.moe_select(z, self.corr, ids, wts, self.groups, self.keep, experts=self.E, score=self.score,
+                       worth=self.group_worth, scale=self.scale, bias=self.br)
         ys = gate = None
         if self.shared is not None:
             ys, _ = self.shared.forward(ctx, h, out="shared_out")

@@ -20,7 +20,7 @@ def tensor_seed(seed, name):
 
 def random_tensors(shapes, seed, dtype=torch.float32, device="cpu", std=0.02, norm_std=0.01, std_by_name=()):
     """shapes: {name: (shape, kind)} with kind "matrix" | "norm" | "bias" | "alpha" (one number about 1) | "depth" (the
-    coefficients of a weighted average) -> {name: tensor of dtype on device}.
+    coefficients of a weighted average) | "fraction" (numbers between 0 and 1) -> {name: tensor of dtype on device}.
     std_by_name: (substring, std) pairs; the first whose substring is in a matrix's or bias's name replaces std."""
     out = {}
     for name, (shape, kind) in shapes.items():
@@ -31,6 +31,8 @@ def random_tensors(shapes, seed, dtype=torch.float32, device="cpu", std=0.02, no
             x = 1.0 + norm_std * x
         elif kind == "depth":               # coefficients of a weighted average: about 1 / their number each
             x = 1.0 / max(1, x.numel()) + norm_std * x
+        elif kind == "fraction":
+            x = torch.sigmoid(x)
         else:
             x = next((s for sub, s in std_by_name if sub in name), std) * x
         out[name] = x.to(dtype)

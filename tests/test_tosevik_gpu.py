@@ -231,7 +231,7 @@ def test_softmax_choice_among_groups(E, top, groups, keep, scale):
     chosen = plain.choose(s, top, groups, keep)
     ids = torch.empty(N, top, dtype=torch.int32, device=DEV)
     wts = torch.empty(N, top, device=DEV)
-    ops.moe_select(z.float().to(DEV), None, ids, wts, groups, keep, experts=E, softmax=True, worth="max", scale=scale)
+    ops.moe_select(z.float().to(DEV), None, ids, wts, groups, keep, experts=E, score="softmax", worth="max", scale=scale)
     ids, wts = ids.cpu().long(), wts.cpu().double()
     assert torch.equal(ids.sort(-1).values, chosen.sort(-1).values)
     assert torch.allclose(wts, scale * s.gather(1, ids), rtol=1e-5, atol=1e-7)

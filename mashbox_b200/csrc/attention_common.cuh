@@ -14,6 +14,7 @@ struct AttnParams {
     float* part_o; float* part_ml; int max_splits;
     int* counters;                          // one per (first item of a split group, kv head), zero between launches; or null
     int H, KV, G, page, num_pages, window;
+    int keep = 0;                           // behind the window the first `keep` positions stay visible (0 without a window)
     int page_shift;                         // log2(page) when the page size is a power of two, else -1
     float scale_log2;
     int* err;
@@ -34,6 +35,19 @@ struct AttnParams {
     // the form of the tcgen05 kernel whose weights are sigmoids: a distance slope and a bias per query head (null: 0)
     const float* sig_slopes = nullptr;
     const float* sig_bias = nullptr;
+};
+
+// The key tiles of BN keys that queries from position lo (the first key their window reaches) to hi - 1 read: `front`
+// tiles of kept first positions, as far as they end before the window's first tile, then the window's.
+struct KeyTiles {
+    int front, skip;
+    __device__ __forceinline__ KeyTiles() {}
+    __device__ __forceinline__ KeyTiles(int keep, int lo, int BN) {
+        front = min((keep + BN - 1) / BN, lo / BN);
+        skip = lo / BN - front;
+    }
+    __device__ __forceinline__ int count(int hi, int BN) const { return (hi + BN - 1) / BN - skip; }
+    __device__ __forceinline__ int key(int t, int BN) const { return (t < front ? t : t + skip) * BN; }      // first key of tile t
 };
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, int bytes) {

@@ -30,7 +30,6 @@ struct GenParams {
     float scale, softcap;                   // softcap 0: none
     const float* sinks;                     // one per query head, or null
     const bf16* gate; int gate_stride;      // gate[n * gate_stride + h], or null
-    int keep;                               // behind the window the first `keep` positions stay visible
 };
 
 // what a finished row is multiplied by and what its denominator gains: the sink joins after every key
@@ -48,7 +47,7 @@ __device__ __forceinline__ void ga_finish(const GenParams& P, int n, int h, floa
 
 template <int HD, int BN>
 __device__ __forceinline__ void load_tile(bf16* dst, const bf16* pool, int row_elems, const AttnParams& P, const int* tb,
-                                          int kvh, int kb, int lo, int hi, int keep, int tid) {
+                                          int kvh, int kb, int lo, int hi, int tid) {
     constexpr int CH = HD / 8;
     const int shift = P.page_shift, mask = P.page - 1;
     int last_block = -1, pg = -1;
@@ -58,7 +57,7 @@ __device__ __forceinline__ void load_tile(bf16* dst, const bf16* pool, int row_e
         const int kp = kb + row;
         const bf16* src = pool;
         int bytes = 0;
-        if ((kp >= lo || kp < keep) && kp < hi) {        // below lo a window may have given the pages back
+        if ((kp >= lo || kp < P.keep) && kp < hi) {        // below lo a window may have given the pages back
             int block, slot;
             if (shift >= 0) { block = kp >> shift; slot = kp & mask; }
             else { block = kp / P.page; slot = kp - block * P.page; }
@@ -101,11 +100,8 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
     const int pos_min = pos0 + row0 / G, pos_max = pos0 + row_last / G;
     const int hi = pos_max + 1;
     const int lo = (P.window > 0 && pos_min - P.window + 1 > 0) ? pos_min - P.window + 1 : 0;
-    const int lo_al = (lo / BN) * BN;
-    // with kept first positions: the tiles that hold them, as far as they end before the window's first tile, come first
-    const int front = min((GP.keep + BN - 1) / BN, lo_al / BN), skip = lo_al / BN - front;
-    const int n_tiles = front + (hi - lo_al + BN - 1) / BN;
-    auto tile_key = [&](int t) { return (t < front ? t : t + skip) * BN; };
+    const KeyTiles tiles(P.keep, lo, BN);
+    const int n_tiles = tiles.count(hi, BN);
     const int tps = (n_tiles + n_splits - 1) / n_splits;
     const int t_begin = split * tps, t_end = min(n_tiles, t_begin + tps);
     const int* tb = P.table + (size_t)P.seq_row[seq] * P.max_blocks;
@@ -123,8 +119,8 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
     cp_async_commit();
     auto fetch = [&](int t) {
         bf16* st = kvs + (size_t)((t - t_begin) % STAGES) * STAGE;
-        load_tile<DK, BN>(st, P.kpool, GP.k_row, P, tb, kvh, tile_key(t), lo, hi, GP.keep, tid);
-        if (!SHARED) load_tile<DV, BN>(st + BN * ROWK, P.vpool, GP.v_row, P, tb, kvh, tile_key(t), lo, hi, GP.keep, tid);
+        load_tile<DK, BN>(st, P.kpool, GP.k_row, P, tb, kvh, tiles.key(t, BN), lo, hi, tid);
+        if (!SHARED) load_tile<DV, BN>(st + BN * ROWK, P.vpool, GP.v_row, P, tb, kvh, tiles.key(t, BN), lo, hi, tid);
     };
 #pragma unroll
     for (int s = 0; s < STAGES - 1; s++) {
@@ -171,7 +167,7 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
         }
         const bf16* kt = kvs + (size_t)((t - t_begin) % STAGES) * STAGE;
         const bf16* vt = SHARED ? kt : kt + BN * ROWK;
-        const int kb = tile_key(t);
+        const int kb = tiles.key(t, BN);
 
         float s[NT][4];
 #pragma unroll
@@ -194,7 +190,7 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const GenParams GP) {
             for (int e = 0; e < 4; e++) {
                 const int i = e >> 1;
                 const int key = kb + nbase + j * 8 + 2 * tig + (e & 1);
-                const bool ok = key <= rpos[i] && (key >= rlo[i] || key < GP.keep);
+                const bool ok = key <= rpos[i] && (key >= rlo[i] || key < P.keep);
                 float v = s[j][e] * GP.scale;
                 // tanh(x) = 1 - 2 / (e^2x + 1) on the fast exponential and division (a few ulp; both ends saturate cleanly):
                 // tanhf's own code was the longest chain of the tile (stalls on fixed-latency waits, tensor pipe 20 %)
@@ -384,7 +380,7 @@ static void ga_fill(GenParams& GP, const void* q, int q_stride, void* out, const
     P.err = err;
     GP.k_row = k_row; GP.v_row = v_row; GP.scale = scale; GP.softcap = softcap; GP.sinks = sinks;
     GP.gate = (const bf16*)gate; GP.gate_stride = gate_stride;
-    GP.keep = window > 0 ? keep : 0;        // without a window every position is visible anyway
+    P.keep = window > 0 ? keep : 0;         // without a window every position is visible anyway
 }
 
 // decode != 0: items are tiles of at most 16 rows; else tiles of 64 rows.

@@ -126,7 +126,8 @@ __device__ __forceinline__ uint64_t umma_desc_join(uint32_t lo) {
 
 // One work unit: 256 packed rows of one sequence and one kv head, as two query tiles, and the key tiles they read.
 struct T5Unit {
-    int kvh, row0, R, G, pos0, tok0, lo, lo_al, T, hi;
+    int kvh, row0, R, G, pos0, tok0, lo, T, hi;
+    KeyTiles keys;
     int T0, T1, pmin0, pmin1, pmax0, pmax1;                         // per query tile: key tiles, first and last position
     const int* tb;
     __device__ __forceinline__ int tiles(int g) const { return g == 0 ? T0 : T1; }
@@ -146,10 +147,10 @@ __device__ __forceinline__ bool t5_unit(const AttnParams& P, int unit, T5Unit& U
 #else
     U.lo = (P.window > 0 && pos_min - P.window + 1 > 0) ? pos_min - P.window + 1 : 0;
 #endif
-    U.lo_al = (U.lo / T5_BN) * T5_BN;
+    U.keys = KeyTiles(P.keep, U.lo, T5_BN);
     U.pmin0 = pos_min;
     U.pmax0 = U.pos0 + (min(U.R, U.row0 + T5_BM) - 1) / U.G;
-    U.T0 = (U.pmax0 + 1 - U.lo_al + T5_BN - 1) / T5_BN;             // at least one
+    U.T0 = U.keys.count(U.pmax0 + 1, T5_BN);                        // at least one
 #ifdef T5_DIFF
     U.pmin1 = U.pmin0; U.pmax1 = U.pmax0; U.T1 = U.T0;             // the second tile is the second map of the same rows
 #else
@@ -157,7 +158,7 @@ __device__ __forceinline__ bool t5_unit(const AttnParams& P, int unit, T5Unit& U
     if (r1 < U.R) {
         U.pmin1 = U.pos0 + r1 / U.G;
         U.pmax1 = U.pos0 + (min(U.R, r1 + T5_BM) - 1) / U.G;
-        U.T1 = (U.pmax1 + 1 - U.lo_al + T5_BN - 1) / T5_BN;
+        U.T1 = U.keys.count(U.pmax1 + 1, T5_BN);
     } else {
         U.pmin1 = U.pmax1 = 0;
         U.T1 = 0;
@@ -245,8 +246,8 @@ __global__ void __launch_bounds__(T5_THREADS, 1) attn_tc5_kernel(const AttnParam
         for (; ok && unit >= 0; k++, unit = t5_unit_at(k, n_units), live = unit >= 0 && t5_unit(P, unit, U)) {
             if (!live) continue;
             auto page_of = [&](int t) -> int {
-                const int key0 = U.lo_al + t * T5_BN + p * page, block = key0 >> shift;
-                const bool live = lane < boxes && key0 < U.hi && key0 + page > U.lo && block < P.max_blocks;
+                const int key0 = U.keys.key(t, T5_BN) + p * page, block = key0 >> shift;
+                const bool live = lane < boxes && key0 < U.hi && (key0 + page > U.lo || key0 < P.keep) && block < P.max_blocks;
                 return live ? __ldg(U.tb + block) : 0;
             };
             // K of tile t+1 goes out before V of tile t: the key stage is free as soon as the score products that read
@@ -259,9 +260,9 @@ __global__ void __launch_bounds__(T5_THREADS, 1) attn_tc5_kernel(const AttnParam
                 if (lane == 0) mbar_expect_tx(fb, TILE);
                 __syncwarp();
                 if (lane < boxes) {
-                    const int key0 = U.lo_al + t * T5_BN + p * page;
+                    const int key0 = U.keys.key(t, T5_BN) + p * page;
                     if (pg < 0 || pg >= P.num_pages) {
-                        if (key0 < U.hi && key0 + page > U.lo) mb_set_error(P.err, pg < 0 ? MB_ERR_PAGE_MISSING : MB_ERR_PAGE_RANGE);
+                        if (key0 < U.hi && (key0 + page > U.lo || key0 < P.keep)) mb_set_error(P.err, pg < 0 ? MB_ERR_PAGE_MISSING : MB_ERR_PAGE_RANGE);
                         pg = 0;                                      // any page: every key of it is masked
                     }
                     const uint32_t dst = (keys ? k_s0 : v_s0) + s * TILE + h * T5_HALF + p * page * 128;
@@ -410,7 +411,8 @@ __global__ void __launch_bounds__(T5_THREADS, 1) attn_tc5_kernel(const AttnParam
 #else
             const int G = U.G, R = U.R, r = U.row0 + g * T5_BM + r_loc;
 #endif
-            const int tok0 = U.tok0, kvh = U.kvh, lo_al = U.lo_al, pos0 = U.pos0;
+            const int tok0 = U.tok0, kvh = U.kvh, pos0 = U.pos0;
+            const KeyTiles keys = U.keys;
             int rpos = -1, rlo = 0;
             if (r < R) {
                 rpos = pos0 + r / G;
@@ -434,13 +436,13 @@ __global__ void __launch_bounds__(T5_THREADS, 1) attn_tc5_kernel(const AttnParam
                 // of the tile before, which read the probabilities in this buffer and wrote the accumulator
                 if (!mbar_wait(s_full0 + 8 * g, (nt + t) & 1, P.err)) { ok = false; break; }
                 tc_fence_after();
-                const int kb = lo_al + t * T5_BN;
+                const int kb = keys.key(t, T5_BN);
 #ifdef T5_DIFF
                 // every key of the tile lies at or before the first row and in the block of positions of the last row
                 // (and so of every row between)
                 const bool full_tile = kb + T5_BN - 1 <= pos_min_g && kb >= ((P.window > 0) ? pos_max_g / P.window * P.window : 0);
 #else
-                const bool full_tile = kb + T5_BN - 1 <= pos_min_g && kb >= ((P.window > 0) ? pos_max_g - P.window + 1 : 0);
+                const bool full_tile = kb + T5_BN - 1 <= pos_min_g && (kb >= ((P.window > 0) ? pos_max_g - P.window + 1 : 0) || kb + T5_BN <= P.keep);
 #endif
                 // the row's 128 scores come from tensor memory with four loads and ONE wait (a load and its wait are a
                 // round trip of several hundred cycles) and stay in registers for both passes
@@ -497,7 +499,7 @@ __global__ void __launch_bounds__(T5_THREADS, 1) attn_tc5_kernel(const AttnParam
 #pragma unroll
                         for (int i = 0; i < 32; i++) {
                             const int key = kb + c * 32 + i;
-                            if (!(key <= rpos && key >= rlo)) sv[c][i] = 0xff800000u;
+                            if (!(key <= rpos && (key >= rlo || key < P.keep))) sv[c][i] = 0xff800000u;
                             mxs[i & 7] = fmaxf(mxs[i & 7], __uint_as_float(sv[c][i]));
                         }
                 }
@@ -744,6 +746,9 @@ MB_API int T5_ENTRY(const void* q, int q_stride, void* out, const void* kpool, c
 #ifdef T5_SIG
                             const float* slopes, const float* bias,             // per query head, or null (0)
 #endif
+#if !defined(T5_DIFF) && !defined(T5_SIG)
+                            int keep,                                           // first positions seen behind the window
+#endif
                             int* err, cudaStream_t st) {
     if (n_items == 0) return 0;
     if (!mb_attn_tc5_supports(HD, page) || KV < 1 || H % KV || KV > 65535) return -2;
@@ -761,6 +766,9 @@ MB_API int T5_ENTRY(const void* q, int q_stride, void* out, const void* kpool, c
     P.table = table; P.max_blocks = max_blocks;
     P.part_o = nullptr; P.part_ml = nullptr; P.max_splits = 1; P.counters = nullptr;
     P.H = H; P.KV = KV; P.G = H / KV; P.page = page; P.num_pages = num_pages; P.window = window;
+#if !defined(T5_DIFF) && !defined(T5_SIG)
+    P.keep = window > 0 ? keep : 0;
+#endif
     P.page_shift = -1;
     for (int sft = 0; sft < 31; sft++) if ((1 << sft) == page) P.page_shift = sft;
     P.scale_log2 = scale * 1.4426950408889634f;

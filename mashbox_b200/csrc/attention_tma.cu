@@ -119,8 +119,8 @@ __global__ void __launch_bounds__(160, 2) attn_tma_kernel(const AttnParams P, co
     const int pos_min = pos0 + row0 / G, pos_max = pos0 + row_last / G;
     const int hi = pos_max + 1;
     const int lo = (P.window > 0 && pos_min - P.window + 1 > 0) ? pos_min - P.window + 1 : 0;
-    const int lo_al = (lo / BN) * BN;
-    const int n_tiles = (hi - lo_al + BN - 1) / BN;
+    const KeyTiles tiles(P.keep, lo, BN);
+    const int n_tiles = tiles.count(hi, BN);
     const int tps = (n_tiles + n_splits - 1) / n_splits;
     const int t_begin = split * tps, t_end = min(n_tiles, t_begin + tps);
     const int* tb = P.table + (size_t)P.seq_row[seq] * P.max_blocks;
@@ -151,8 +151,8 @@ __global__ void __launch_bounds__(160, 2) attn_tma_kernel(const AttnParams P, co
         const int p = b / HALVES, h = b % HALVES;
         const bool active = lane < 2 * boxes;
         auto page_of = [&](int t) -> int {
-            const int key0 = lo_al + t * BN + p * page, block = key0 >> shift;
-            const bool live = active && key0 < hi && key0 + page > lo && block < P.max_blocks;
+            const int key0 = tiles.key(t, BN) + p * page, block = key0 >> shift;
+            const bool live = active && key0 < hi && (key0 + page > lo || key0 < P.keep) && block < P.max_blocks;
             return live ? __ldg(tb + block) : 0;
         };
         int pg = (t_begin < t_end) ? page_of(t_begin) : 0;
@@ -165,9 +165,9 @@ __global__ void __launch_bounds__(160, 2) attn_tma_kernel(const AttnParams P, co
             if (lane == 0) mbar_expect_tx(fb, 2u * TILE * 2u);
             __syncwarp();
             if (active) {
-                const int key0 = lo_al + t * BN + p * page;
+                const int key0 = tiles.key(t, BN) + p * page;
                 if (pg < 0 || pg >= P.num_pages) {
-                    if (key0 < hi && key0 + page > lo) mb_set_error(P.err, pg < 0 ? MB_ERR_PAGE_MISSING : MB_ERR_PAGE_RANGE);
+                    if (key0 < hi && (key0 + page > lo || key0 < P.keep)) mb_set_error(P.err, pg < 0 ? MB_ERR_PAGE_MISSING : MB_ERR_PAGE_RANGE);
                     pg = 0;                                            // any page: every key of it is masked
                 }
                 const uint32_t dst = smem_u32(kvs + (size_t)s * 2 * TILE) + which * TILE * 2 +
@@ -268,7 +268,7 @@ __global__ void __launch_bounds__(160, 2) attn_tma_kernel(const AttnParams P, co
         if (!mbar_wait(full0 + 8 * s, round & 1, P.err)) return;
         const bf16* kt = kvs + (size_t)s * 2 * TILE;
         const bf16* vt = kt + TILE;
-        const int kb = lo_al + t * BN;
+        const int kb = tiles.key(t, BN);
         if (ROPE && DECODE && t == n_tiles - 1 && pos0 - kb >= nbase && pos0 - kb < nbase + 16) {
             // the token's own slot is among this warp's keys of the tile: its new key and value rows go in
             const int rowk = pos0 - kb;
@@ -295,7 +295,7 @@ __global__ void __launch_bounds__(160, 2) attn_tma_kernel(const AttnParams P, co
         }
         // a tile whose keys every row of the block may read needs no mask (all tiles but the last and, with a window,
         // the first ones); rows past the end of the block then get finite scores, and they are never written
-        const bool full_tile = kb + BN - 1 <= pos_min && kb >= ((P.window > 0) ? pos_max - P.window + 1 : 0);
+        const bool full_tile = kb + BN - 1 <= pos_min && (kb >= ((P.window > 0) ? pos_max - P.window + 1 : 0) || kb + BN <= P.keep);
         float tmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int j = 0; j < NT; j++) {
@@ -305,7 +305,7 @@ __global__ void __launch_bounds__(160, 2) attn_tma_kernel(const AttnParams P, co
                 float v = sc[j][e] * P.scale_log2;
                 if (!full_tile) {
                     const int key = kb + nbase + j * 8 + 2 * tig + (e & 1);
-                    if (!(key <= rpos[ii] && key >= rlo[ii])) v = -INFINITY;
+                    if (!(key <= rpos[ii] && (key >= rlo[ii] || key < P.keep))) v = -INFINITY;
                 }
                 sc[j][e] = v;
                 tmax[ii] = fmaxf(tmax[ii], v);
@@ -628,7 +628,7 @@ static int attn_tma_run(const void* q, int q_stride, void* out, const void* kpoo
                         const int* pos0, const int* part_base, const int* seq_row, const int* table, int max_blocks,
                         float* part_o, float* part_ml, int max_splits, int H, int KV, int HD, int page, int num_pages,
                         int window, float scale, int* counters, int* err, cudaStream_t st, int fuse, const float* bias,
-                        const float* freqs, int RD, int pairing, int cluster = 0) {
+                        const float* freqs, int RD, int pairing, int cluster = 0, int keep = 0) {
     if (n_items == 0) return 0;
     if (cluster > 1 && (!decode || cluster > 8)) return -2;
     if (!mb_attn_tma_supports(HD, page) || KV < 1 || H % KV || KV > 65535) return -2;
@@ -641,6 +641,7 @@ static int attn_tma_run(const void* q, int q_stride, void* out, const void* kpoo
     P.table = table; P.max_blocks = max_blocks;
     P.part_o = part_o; P.part_ml = part_ml; P.max_splits = max_splits; P.counters = counters;
     P.H = H; P.KV = KV; P.G = H / KV; P.page = page; P.num_pages = num_pages; P.window = window;
+    P.keep = window > 0 ? keep : 0;
     P.page_shift = -1;
     for (int sft = 0; sft < 31; sft++) if ((1 << sft) == page) P.page_shift = sft;
     P.scale_log2 = scale * 1.4426950408889634f;
@@ -665,10 +666,10 @@ MB_API int mb_attn_tma_bf16(const void* q, int q_stride, void* out, const void* 
                             const void* items, int n_items, int decode, const int* q_start, const int* q_len,
                             const int* pos0, const int* part_base, const int* seq_row, const int* table, int max_blocks,
                             float* part_o, float* part_ml, int max_splits, int H, int KV, int HD, int page, int num_pages,
-                            int window, float scale, int* counters, int* err, cudaStream_t st) {
+                            int window, int keep, float scale, int* counters, int* err, cudaStream_t st) {
     return attn_tma_run(q, q_stride, out, kpool, vpool, items, n_items, decode, q_start, q_len, pos0, part_base, seq_row,
                         table, max_blocks, part_o, part_ml, max_splits, H, KV, HD, page, num_pages, window, scale,
-                        counters, err, st, 0, nullptr, nullptr, 0, 0);
+                        counters, err, st, 0, nullptr, nullptr, 0, 0, 0, keep);
 }
 
 // The decode form for a step in which every sequence brings one token, with the rotate-and-store step folded in: qkv
@@ -677,12 +678,12 @@ MB_API int mb_attn_tma_bf16(const void* q, int q_stride, void* out, const void* 
 MB_API int mb_attn_tma_rope_bf16(const void* qkv, int q_stride, void* out, void* kpool, void* vpool, const void* items,
                                  int n_items, const int* q_start, const int* q_len, const int* pos0, const int* part_base,
                                  const int* seq_row, const int* table, int max_blocks, float* part_o, float* part_ml,
-                                 int max_splits, int H, int KV, int HD, int page, int num_pages, int window, float scale,
+                                 int max_splits, int H, int KV, int HD, int page, int num_pages, int window, int keep, float scale,
                                  int* counters, int* err, const float* bias, const float* freqs, int RD, int pairing,
                                  cudaStream_t st) {
     return attn_tma_run(qkv, q_stride, out, kpool, vpool, items, n_items, 1, q_start, q_len, pos0, part_base, seq_row, table,
                         max_blocks, part_o, part_ml, max_splits, H, KV, HD, page, num_pages, window, scale, counters,
-                        err, st, 1, bias, freqs, RD, pairing);
+                        err, st, 1, bias, freqs, RD, pairing, 0, keep);
 }
 
 // The decode form launched as thread-block clusters: every sequence of the launch is cut into `cluster` splits (2 to
@@ -692,12 +693,12 @@ MB_API int mb_attn_tma_rope_bf16(const void* qkv, int q_stride, void* out, void*
 MB_API int mb_attn_tma_cluster_bf16(const void* q, int q_stride, void* out, void* kpool, void* vpool, const void* items,
                                     int n_items, const int* q_start, const int* q_len, const int* pos0, const int* seq_row,
                                     const int* table, int max_blocks, int cluster, int H, int KV, int HD, int page,
-                                    int num_pages, int window, float scale, int* err, int rope, const float* bias,
+                                    int num_pages, int window, int keep, float scale, int* err, int rope, const float* bias,
                                     const float* freqs, int RD, int pairing, cudaStream_t st) {
     if (cluster < 2) return -2;
     return attn_tma_run(q, q_stride, out, kpool, vpool, items, n_items, 1, q_start, q_len, pos0, nullptr, seq_row, table,
                         max_blocks, nullptr, nullptr, cluster, H, KV, HD, page, num_pages, window, scale, nullptr, err, st,
-                        rope, bias, freqs, RD, pairing, cluster);
+                        rope, bias, freqs, RD, pairing, cluster, keep);
 }
 
 static int attn_tma_query(int HD, int rope, int what) {

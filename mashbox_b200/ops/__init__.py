@@ -1267,8 +1267,9 @@ def attention_tma_active_clusters(HD, cluster):
 
 def attention_tma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_start, q_len, pos0, part_base, seq_row,
                   table, part_o, part_ml, max_splits, H, KV, HD, page, num_pages, window, scale, err, merge=False,
-                  rope=None, cluster=0):
+                  rope=None, cluster=0, keep=0):
     """The same contract as attention_mma, with K/V tiles loaded by TMA (head sizes 64 and 128, pages of 8 to 64).
+    keep: behind the window the first `keep` positions stay visible.
     merge: the last block of every split group merges the group's partial results and writes `out`, so no
     attention_merge is needed afterwards (only when attention_tma_merges(n_items, KV)).
     cluster = n > 1 (decode form): every sequence of the launch is cut into n splits and the blocks of a sequence and kv
@@ -1285,9 +1286,9 @@ def attention_tma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_star
         _cuda(bias, freqs)
         f = _fn("attention_tma", "mb_attn_tma_cluster_bf16",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                 c_void_p, c_int] + [c_int] * 7 + [c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
+                 c_void_p, c_int] + [c_int] * 8 + [c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
         code = f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, _p(q_start), _p(q_len), _p(pos0),
-                 _p(seq_row), _p(table), table.shape[1], int(cluster), H, KV, HD, page, num_pages, window or 0,
+                 _p(seq_row), _p(table), table.shape[1], int(cluster), H, KV, HD, page, num_pages, window or 0, int(keep),
                  float(scale), _p(err), 1 if rope is not None else 0, _p(bias), _p(freqs), int(RD), int(pairing), _stream())
         if code == -6:
             raise KernelError("attention_tma: the driver refused the tensor map of the cache pool")
@@ -1309,19 +1310,19 @@ def attention_tma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_star
         _cuda(bias, freqs)
         f = _fn("attention_tma", "mb_attn_tma_rope_bf16",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                 c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 7 + [c_float, c_void_p, c_void_p, c_void_p,
+                 c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_void_p, c_void_p, c_void_p,
                                                                                 c_void_p, c_int, c_int, c_void_p])
         code = f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, _p(q_start), _p(q_len), _p(pos0),
                  _p(part_base), _p(seq_row), _p(table), table.shape[1], _p(part_o), _p(part_ml), max_splits, H, KV, HD,
-                 page, num_pages, window or 0, float(scale), _p(counters), _p(err), _p(bias), _p(freqs), int(RD),
+                 page, num_pages, window or 0, int(keep), float(scale), _p(counters), _p(err), _p(bias), _p(freqs), int(RD),
                  int(pairing), _stream())
     else:
         f = _fn("attention_tma", "mb_attn_tma_bf16",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                 c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 7 + [c_float, c_void_p, c_void_p, c_void_p])
+                 c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_void_p, c_void_p, c_void_p])
         code = f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, 1 if decode else 0, _p(q_start),
                  _p(q_len), _p(pos0), _p(part_base), _p(seq_row), _p(table), table.shape[1], _p(part_o), _p(part_ml),
-                 max_splits, H, KV, HD, page, num_pages, window or 0, float(scale), _p(counters), _p(err), _stream())
+                 max_splits, H, KV, HD, page, num_pages, window or 0, int(keep), float(scale), _p(counters), _p(err), _stream())
     if code == -6:
         raise KernelError("attention_tma: the driver refused the tensor map of the cache pool")
     _check(code, "attention_tma")
@@ -1339,15 +1340,15 @@ def attention_tc5_rows():
 
 
 def attention_tc5(q, q_stride, out, kpool, vpool, items, n_items, q_start, q_len, pos0, seq_row, table, H, KV, HD, page,
-                  num_pages, window, scale, err):
+                  num_pages, window, scale, err, keep=0):
     """Prompt-form attention on tcgen05: items are (sequence, tile of attention_tc5_rows() packed rows, 0, 1); head
-    sizes 64 and 128."""
+    sizes 64 and 128.  keep: behind the window the first `keep` positions stay visible."""
     _cuda(q, out, kpool, vpool, items, q_start, q_len, pos0, seq_row, table)
     f = _fn("attention_tc5", "mb_attn_tc5_bf16",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-             c_void_p, c_int] + [c_int] * 6 + [c_float, c_void_p, c_void_p])
+             c_void_p, c_int] + [c_int] * 6 + [c_float, c_int, c_void_p, c_void_p])
     _check(f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, _p(q_start), _p(q_len), _p(pos0),
-             _p(seq_row), _p(table), table.shape[1], H, KV, HD, page, num_pages, window or 0, float(scale),
+             _p(seq_row), _p(table), table.shape[1], H, KV, HD, page, num_pages, window or 0, float(scale), int(keep),
              _p(err), _stream()), "attention_tc5")
 
 

@@ -57,9 +57,10 @@ class PagedAttention:
         """vdim: the width of a value when it is not the key's (the result is heads * vdim wide); softcap: scores become
         softcap tanh(s / softcap); sinks: attend() is handed one number per query head that joins the softmax's
         denominator without a value; gated: attend() is handed a gate per token and query head (the head's result
-        times its sigmoid); keep_first: behind the window the first `keep_first` positions stay visible.  Any of
-        the five, or pools whose rows are wider than what is read of them, make the
-        attention *general*: it runs on the kernels that take all of that."""
+        times its sigmoid).  Any of the four, or pools whose rows are wider than what is read of them, make the
+        attention *general*: it runs on the kernels that take all of that.  keep_first: behind the window the first
+        `keep_first` positions stay visible, which the TMA and tcgen05 kernels take and the general ones; where a step
+        would run another kernel the attention is general too (`is_general`)."""
         self.H, self.KV, self.HD = int(heads), int(kv_heads), int(head_dim)
         if self.H % self.KV:
             raise ConfigError(f"{heads} heads do not divide into {kv_heads} kv heads")
@@ -68,12 +69,21 @@ class PagedAttention:
         self.VD = int(vdim) if vdim else self.HD
         self.softcap = float(softcap) if softcap else None
         self.keep = int(keep_first) if self.window else 0       # without a window every position is visible anyway
-        self.general = self.VD != self.HD or self.softcap is not None or bool(sinks) or bool(gated) or self.keep > 0
+        self.general = self.VD != self.HD or self.softcap is not None or bool(sinks) or bool(gated)
 
     # ------------------------------------------------------------------------------------------ planning
+    def is_general(self, ctx):
+        """whether this step runs the general kernels"""
+        import torch
+        if self.general or not self.keep:
+            return self.general
+        page = ctx.cache.page_size
+        return not (ctx.dtype == torch.bfloat16 and ctx.options.get("attention_kernel", "tma") == "tma"
+                    and ctx.ops.attention_tma_supports(self.HD, page) and not ctx.options.get("plain_attention", False))
+
     def uses_mma(self, ctx):
         import torch
-        if self.general:        # keys and values of their own widths, caps, sinks, gates: the general tensor-core form
+        if self.is_general(ctx):        # keys and values of their own widths, caps, sinks, gates: the general tensor-core form
             return (ctx.dtype == torch.bfloat16 and ctx.ops.attention_general_mma_supports(self.HD, self.VD)
                     and not ctx.options.get("plain_attention", False))
         return ctx.dtype == torch.bfloat16 and ctx.ops.attention_mma_supports(self.HD) and not ctx.options.get(
@@ -82,12 +92,12 @@ class PagedAttention:
     def uses_tc5(self, ctx):
         """prompt-form tiles go to the tcgen05 kernel (its own number of packed rows per block, no splits) when it takes
         the sizes"""
-        return (not self.general and ctx.options.get("attention_prefill_kernel", "tc5") == "tc5"
+        return (not self.is_general(ctx) and ctx.options.get("attention_prefill_kernel", "tc5") == "tc5"
                 and ctx.ops.attention_tc5_supports(self.HD, ctx.cache.page_size))
 
     def _tma(self, ctx):
         """decode-form sequences go to the TMA kernel (whose splits may meet in a cluster)"""
-        return (not self.general and ctx.options.get("attention_kernel", "tma") == "tma"
+        return (not self.is_general(ctx) and ctx.options.get("attention_kernel", "tma") == "tma"
                 and ctx.ops.attention_tma_supports(self.HD, ctx.cache.page_size))
 
     def plan_key(self):
@@ -203,7 +213,7 @@ class PagedAttention:
         ops = ctx.ops
         H, KV, HD = self.H, self.KV, self.HD
         page, pages = ctx.cache.page_size, ctx.cache.pool_pages
-        if self.general:
+        if self.is_general(ctx):
             self.attend_general(ctx, qkv, width, out, table, kpool, vpool, sinks, gate)
             return
         if self.uses_mma(ctx):
@@ -221,19 +231,21 @@ class PagedAttention:
             fused = (tma and n_part > 0 and ctx.options.get("attention_fused_merge", True)
                      and ops.attention_tma_merges(max(plan["n_pre"], plan["n_mid"], plan["n_dec"]), KV))
             extra = dict(merge=True) if fused else {}
+            if self.keep:
+                extra["keep"] = self.keep
             if rope is not None:
                 extra["rope"] = rope
             if plan["tc5"] and plan["n_pre"]:
                 ops.attention_tc5(qkv, width, out, kpool, vpool, ctx.dev(nm + "pre"), plan["n_pre"], ctx.dev("q_start"),
                                   ctx.dev("q_len"), ctx.dev("pos0"), ctx.dev("seq_row"), table, H, KV, HD, page, pages,
-                                  self.window, self.scale, ctx.err)
+                                  self.window, self.scale, ctx.err, keep=self.keep)
             for form, n_items, decode in ((nm + "pre", 0 if plan["tc5"] else plan["n_pre"], False),
                                           (nm + "mid", plan["n_mid"], False), (nm + "dec", plan["n_dec"], True)):
                 if n_items and decode and plan["cluster"]:
                     ops.attention_tma(qkv, width, out, kpool, vpool, ctx.dev(form), n_items, True, ctx.dev("q_start"),
                                       ctx.dev("q_len"), ctx.dev("pos0"), None, ctx.dev("seq_row"), table, None, None, 1,
                                       H, KV, HD, page, pages, self.window, self.scale, ctx.err,
-                                      rope=extra.get("rope"), cluster=plan["cluster"])
+                                      rope=extra.get("rope"), cluster=plan["cluster"], keep=self.keep)
                 elif n_items:
                     flash(qkv, width, out, kpool, vpool, ctx.dev(form), n_items, decode, ctx.dev("q_start"),
                           ctx.dev("q_len"), ctx.dev("pos0"), ctx.dev(nm + "part_base"), ctx.dev("seq_row"),
@@ -400,7 +412,6 @@ class GatedAttention(PagedAttention):
                  sink=None, gate=False, position=None, window=None, keep_first=0, value_mix=None, prefix="", names=None):
         super().__init__(heads, kv_heads, head_dim, window, scale, vdim=vdim, softcap=softcap, sinks=sink is not None,
                          gated=gate, keep_first=keep_first)
-        self.general = True         # this mixer's own path: separate key and value pools, q/k norms
         self.D, self.eps, self.sink, self.gate = int(hidden), float(eps), sink, bool(gate)
         if qk_norm not in (True, False, None, "after") or value_mix not in (None, "keep", "mix"):
             raise ConfigError(f"this attention has no q/k norm {qk_norm!r} or value mixing {value_mix!r}")

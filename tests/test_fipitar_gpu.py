@@ -230,7 +230,8 @@ def test_head_norms_rotation_and_cache_write(dtype, H, KV, DK, DV, RD, pairing, 
     r = dev(rows, dtype)
     err = torch.zeros(1, dtype=torch.int32, device=DEV)
     ops.norm_rope_kv_write(r, dev(qw) if normed else None, dev(kw) if normed else None, 1e-6, dev(freqs) if RD else None, RD,
-                           pairing, gain, i32(positions), i32(tok_row), i32(table), kpool, vpool, H, KV, DK, DV, page, pages, err)
+                           pairing, gain, i32(positions), i32(tok_row), i32(table), kpool, vpool, H, KV, DK, DV, page, pages, err,
+                           norm="before" if normed else None)
     assert int(err.item()) == 0
 
     def want_heads(x, w):

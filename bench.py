@@ -763,6 +763,183 @@ def fipitar_configs(size, layers, vocab=32000, context=8192):
     return fp, sf
 
 
+# Layer sizes for `--design pobelorn`: attention (a window of 4,096 positions with 64 kept first tokens, heads of 128 x 128 of
+# which half a head is rotated, a kv head to four query heads, values mixed) in the first and last layer of a run of four,
+# lightning attention (heads of 128 x 128) between them, routed experts with a shared expert in every layer.  The Tosevik
+# decoder beside it -- the closest design the engine has: the same recurrence in three layers of four, attention over cached
+# keys beside it in the fourth, routed experts with a shared one -- has the same width, layers, heads, head sizes and experts.
+POBELORN_SIZES = {k: dict(v, window=4096, keep_first=64) for k, v in TOSEVIK_SIZES.items()}
+
+
+def pobelorn_configs(size, layers, vocab=32000, context=8192):
+    from mashbox_b200.config import pobelorn as F
+    z = POBELORN_SIZES[size]
+    D, H, dim = z["width"], z["heads"], z["dim"]
+    att = F.AttentionMixer(heads=H, kv_heads=max(1, H // 4), dim=dim, vdim=dim, scale=dim ** -0.5, window=z["window"],
+                           keep_first=z["keep_first"], v_mix=True, rot=F.Rotation(dim // 2, 500000.0, (4.0, 2048.0, 32.0, 1.0)))
+    li = F.LightningMixer(heads=H, dim=dim, vdim=dim, decay=tuple(1.0 - 2.0 ** (-5.0 - 3.0 * h / max(1, H - 1)) for h in range(H)))
+    moe = F.ExpertsFF(ff=z["ff"], experts=z["experts"], top=z["top"], shared_ff=z["shared"])
+    pb = F.PobelornConfig("Pobelorn", width=D, vocab=vocab, norm_eps=1e-6, embedding_scale=1.0, layers=tuple(
+        F.PobelornLayer("attention", att, moe) if i % 4 in (0, 3) else F.PobelornLayer("lightning", li, moe)
+        for i in range(layers)))
+    return pb, tosevik_configs(size, layers, vocab, context)[0]
+
+
+def pobelorn_kernels(a, z, P, B, ctx, pk):
+    """The kernels of the Pobelorn decoder, each beside the like kernel of the Tosevik (or Llama, or Fipitar) decoder at
+    equal sizes: CUDA-event time of single launches after an L2 flush, and the fraction of the measured peak that the
+    algorithmic bytes (copy bandwidth) or FLOPs (bf16 tensor throughput) come to."""
+    import torch
+    from mashbox_b200 import ops
+    from mashbox_b200.parts.attention import PagedAttention
+    dev = "cuda:0"
+    D, H, dim, F, E, top = (z[k] for k in ("width", "heads", "dim", "ff", "experts", "top"))
+    page, win, keep = 16, z["window"], z["keep_first"]
+    KV = max(1, H // 4)
+    gen = torch.Generator(device=dev).manual_seed(0)
+    bf = lambda *s: (torch.randn(*s, generator=gen, device=dev) * 0.5).to(torch.bfloat16)
+    f32 = lambda *s: torch.randn(*s, generator=gen, device=dev) * 0.5
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    err = ops.new_error_word(dev)
+
+    def timed(f):
+        for _ in range(3):
+            f()
+        ts = []
+        for _ in range(max(5, a.steps // 4)):
+            flush.zero_()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            f()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) * 1e3)
+        return statistics.median(ts)
+
+    mem = lambda us, nbytes: {"us": us, "gbs": nbytes / us / 1e3, "frac_of_copy_peak": nbytes / us / 1e3 / pk["hbm_gbs"]}
+    mat = lambda us, flops: {"us": us, "tflops": flops / us / 1e6, "frac_of_bf16_peak": flops / us / 1e6 / pk["bf16_tflops"]}
+    res = {}
+    # ---- the recurrence (one kernel for lightning attention and retention), and what stands around it in either
+    decay = torch.tensor([1.0 - 2.0 ** (-5.0 - 3.0 * h / max(1, H - 1)) for h in range(H)], device=dev)
+    for form, N, S in (("prompt", P, 1), ("decode", B, B)):
+        C = H * dim
+        q, k, v, o = f32(N, C), f32(N, C) * dim ** -0.5, f32(N, C), f32(N, C)
+        state = torch.zeros(S, C * dim, device=dev)
+        seq = (i32([i * (N // S) for i in range(S)]), i32([N // S] * S), i32(list(range(S))))
+        chunked = ops.retention_splits(N, S, H, dim)
+        us = timed(lambda: ops.retention(q, k, v, decay, o, state, seq, H, dim, dim, chunked=chunked))
+        res[f"recurrence_{form}"] = dict(mem(us, 2 * S * C * dim * 4 + N * C * 4 * 4), form="split" if chunked else "scan")
+        rows, freqs, pos = bf(N, 4 * C), torch.rand(dim // 2, generator=gen, device=dev), torch.arange(N, dtype=torch.int32, device=dev)
+        us = timed(lambda: ops.silu_rows(rows, q, k, v))
+        res[f"lightning_activations_{form}"] = mem(us, N * C * 3 * (2 + 4))
+        us = timed(lambda: ops.retention_prep(rows, 0, C, 2 * C, pos, freqs, q, k, v, H, dim, dim, dim, dim ** -0.5))
+        res[f"retention_prep_tosevik_{form}"] = mem(us, N * C * 3 * (2 + 4))
+        gated, w = torch.empty(N, C, device=dev, dtype=torch.bfloat16), f32(C)
+        us = timed(lambda: ops.gated_rms(o, rows[:, 3 * C:], w, gated, 1, C, 1e-6))
+        res[f"lightning_norm_gate_{form}"] = mem(us, N * C * (4 + 2 + 2))
+        us = timed(lambda: ops.gated_rms(o, rows[:, 3 * C:], None, gated, H, dim, 1e-6, silu=True))
+        res[f"retention_norm_gate_tosevik_{form}"] = mem(us, N * C * (4 + 2 + 2))
+    # ---- attention: a prompt of P tokens; a portion of P tokens far behind the window; B tokens decoded at ctx.  Beside
+    #      Llama's over as many keys; and with values half as wide, on the general kernel, beside Fipitar's
+    own, llama = PagedAttention(H, KV, dim, win, keep_first=keep), PagedAttention(H, KV, dim)
+    narrow = PagedAttention(H, KV, dim, win, keep_first=keep, vdim=dim // 2)
+    fip = PagedAttention(H, KV, dim, None, vdim=dim // 2, softcap=30.0, sinks=True)
+    sinks = f32(H)
+    for name, core in (("attention", own), ("attention_llama", llama), ("attention_narrow_values", narrow),
+                       ("attention_fipitar", fip)):
+        wv = core.VD
+        for form, N, S, end in (("prompt", P, 1, P), ("portion", P, 1, max(ctx, win + P)), ("decode", B, B, ctx)):
+            pairs = min(win + keep, ctx)        # keys a query sees far from the start; the others are given as many
+            if form != "prompt" and not core.window:
+                end = pairs if form == "decode" else pairs + P // 2
+            pages = S * -(-end // page)
+            table = torch.arange(pages, dtype=torch.int32, device=dev).reshape(S, -1)
+            kp, vp = bf(pages, KV, page, dim), bf(pages, KV, page, wv)
+            q, o = bf(N, H * dim), torch.empty(N, H * wv, device=dev, dtype=torch.bfloat16)
+            q_len = [N // S] * S
+            ctx_ = _PlanContext(ops, dev, q_len, [end - n for n in q_len], page, pages, err)
+            core.prepare(ctx_)
+            ctx_.inputs.upload()
+            extra = dict(sinks=sinks) if core is fip else {}
+            us = timed(lambda: core.attend(ctx_, q, H * dim, o, table, kp, vp, **extra))
+            if form == "decode":
+                res[f"{name}_{form}"] = mem(us, S * pairs * KV * (dim + wv) * 2 + N * H * (dim + wv) * 2)
+            else:
+                res[f"{name}_{form}"] = mat(us, 2 * H * (dim + wv) * P * (P / 2 if form == "prompt" else pairs))
+            del kp, vp
+    # ---- heads between the product and attention: rotation, norm, values mixed, cache write; Llama's rotation and write
+    for form, N in (("prompt", P), ("decode", B)):
+        rows = bf(N, (H + 2 * KV) * dim)
+        pages = -(-N // page)
+        table = torch.arange(pages, dtype=torch.int32, device=dev).reshape(1, -1)
+        kp, vp, first = bf(pages, KV, page, dim), bf(pages, KV, page, dim), bf(N, KV * dim)
+        pos, row = torch.arange(N, dtype=torch.int32, device=dev), torch.zeros(N, dtype=torch.int32, device=dev)
+        fr = torch.rand(dim // 2, generator=gen, device=dev)
+        nbytes = 2 * N * (H + 2 * KV) * dim * 2
+        us = timed(lambda: ops.norm_rope_kv_write(rows, None, None, 1e-6, fr, dim // 2, 0, 1.1, pos, row, table, kp, vp, H, KV, dim,
+                                                  dim, page, pages, err, norm="after", v_first=first, lam=0.3))
+        res[f"heads_{form}"] = mem(us, nbytes + N * KV * dim * 2)
+        us = timed(lambda: ops.rope_kv_write(rows, None, pos, row, table, kp, vp, fr, H, KV, dim, dim // 2, 0, page, pages, err))
+        res[f"heads_llama_{form}"] = mem(us, nbytes)
+    # ---- the experts (one set of kernels for both designs), the choice; the dense unit beside SwiGLU of as many weights
+    wg, wu, wd = bf(E, F, D), bf(E, F, D), bf(E, D, F)
+    Fd = (F * top + z["shared"]) // 2 // 16 * 16            # a dense unit with two matrices against SwiGLU's three
+    for form, N in (("prompt", P), ("decode", B)):
+        h = bf(N, D)
+        ids = torch.stack([torch.randperm(E, generator=gen, device=dev)[:top] for _ in range(N)]).int().contiguous()
+        wts, shared, gate = torch.rand(N, top, generator=gen, device=dev), bf(N, D), f32(N, 1)
+        touched = len(set(ids.flatten().tolist()))
+        out = torch.empty(N, D, device=dev, dtype=torch.bfloat16)
+        for name, g_ in (("experts", None), ("experts_tosevik", gate)):
+            if form == "prompt":
+                T = ops.moe_tc5_tiles(N, top, E)
+                rows, act2 = torch.empty(128 * T, D, device=dev, dtype=torch.bfloat16), torch.empty(128 * T, F, device=dev, dtype=torch.bfloat16)
+                y2, places = torch.empty(128 * T, D, device=dev), torch.empty(N * top + T, dtype=torch.int32, device=dev)
+                wgu2 = torch.cat([wg, wu], 1).contiguous()
+                us = timed(lambda: ops.moe_tc5(h, ids, wts, wgu2, wd, out, rows, act2, y2, places, float("inf"), 1.0, 0.0, shared, g_))
+                res[f"{name}_prompt"] = mat(us, 2 * N * top * 3 * F * D)
+                need = max(2 * N * top * 3 * F * D / (pk["bf16_tflops"] * 1e6), touched * 3 * F * D * 2 / (pk["hbm_gbs"] * 1e3))
+                res[f"{name}_prompt"].update(frac_of_roofline=need / us)
+                del wgu2, rows, act2, y2
+            else:
+                y = torch.empty(N, top, D, device=dev)
+                us = timed(lambda: (ops.moe_experts(h, ids, wg, wu, wd, y, float("inf"), 1.0, None, 0.0), ops.moe_combine(y, wts, out, shared, g_)))
+                res[f"{name}_decode"] = dict(mem(us, touched * 3 * F * D * 2), experts_touched=touched)
+        zl, bias = f32(N, E), f32(E)
+        idc, wtc = torch.empty(N, top, dtype=torch.int32, device=dev), torch.empty(N, top, device=dev)
+        res[f"choice_{form}"] = {"us": timed(lambda: ops.moe_select(zl, None, idc, wtc, experts=E, score="softmax_chosen", bias=bias))}
+        res[f"choice_tosevik_{form}"] = {"us": timed(lambda: ops.moe_select(zl, None, idc, wtc, z["groups"], z["keep"], experts=E,
+                                                                           score="softmax", worth="max", scale=2.5))}
+        up, down, act = bf(3 * Fd, D), bf(D, 3 * Fd), torch.empty(N, 3 * Fd, device=dev, dtype=torch.bfloat16)
+        wgu, wdn, a1 = bf(4 * Fd, D), bf(D, 2 * Fd), torch.empty(N, 2 * Fd, device=dev, dtype=torch.bfloat16)
+        if form == "prompt":
+            us = timed(lambda: ops.linear_relu2(h, up, act))
+            res["dense_up_prompt"] = mat(us, 2 * N * 3 * Fd * D)
+            us = timed(lambda: ops.linear_swiglu(h, wgu, a1))
+            res["dense_gate_up_llama_prompt"] = mat(us, 2 * N * 4 * Fd * D)
+            us = timed(lambda: ops.relu2(act, act))
+            res["relu2_rows_prompt"] = mem(us, N * 3 * Fd * 4)
+        else:
+            if ops.fused_relu2_supports(N, 3 * Fd, D, torch.bfloat16):
+                us = timed(lambda: (ops.linear_relu2(h, up, act), ops.linear(act, down, out=out)))
+            else:
+                us = timed(lambda: (ops.linear(h, up, out=act), ops.relu2(act, act), ops.linear(act, down, out=out)))
+            res["dense_decode"] = mem(us, 6 * Fd * D * 2)
+            us = timed(lambda: (ops.linear_swiglu(h, wgu, a1) if ops.fused_swiglu_supports(N, 2 * Fd, D) else
+                                ops.linear_stream(h, wgu, a1, "swiglu"), ops.linear(a1, wdn, out=out)))
+            res["dense_llama_decode"] = mem(us, 6 * Fd * D * 2)
+        del up, down, wgu, wdn
+    # ---- the stream: two outputs added and one norm; Llama's add + norm
+    for form, N in (("prompt", P), ("decode", B)):
+        x, d1, d2, w, nrm = f32(N, D), bf(N, D), bf(N, D), f32(D), torch.empty(N, D, device=dev, dtype=torch.bfloat16)
+        us = timed(lambda: ops.add_rmsnorm_pair(x, d1, d2, w, None, 1e-6, nrm))
+        res[f"add_two_norm_{form}"] = mem(us, N * D * (4 + 4 + 2 + 2 + 2))
+        us = timed(lambda: ops.add_rmsnorm(x, d1, None, w, 1e-6, nrm))
+        res[f"add_norm_llama_{form}"] = mem(us, N * D * (4 + 4 + 2 + 2))
+    return res
+
+
 def fipitar_kernels(a, z, P, B, ctx, pk):
     """The kernels of the Fipitar decoder, each beside the like kernel of the Sufopel (or Llama) decoder at equal sizes:
     CUDA-event time of single launches after an L2 flush, and the fraction of the measured peak that the algorithmic bytes
@@ -905,7 +1082,11 @@ def run_design(a):
     layers = a.layers or 4
     design = a.design
     other = "llama"
-    if design == "fipitar":
+    if design == "pobelorn":
+        z, other = POBELORN_SIZES[a.size], "tosevik"
+        cfgs = dict(zip((design, other), pobelorn_configs(a.size, layers, context=a.context)))
+        single_kernels = pobelorn_kernels
+    elif design == "fipitar":
         z, other = FIPITAR_SIZES[a.size], "sufopel"
         cfgs = dict(zip((design, other), fipitar_configs(a.size, layers, context=a.context)))
         single_kernels = fipitar_kernels
@@ -1457,8 +1638,9 @@ def main():
     ap.add_argument("--requests", type=int, default=0, help="workloads: fewer requests than the workload names")
     ap.add_argument("--pool-tokens", type=int, default=0, help="workloads: size of the cache pool (0: every request fits)")
     ap.add_argument("--seed", type=int, default=0)
-    ap.add_argument("--design", default="", choices=("", "luzosun", "sufopel", "tosevik", "fipitar"),
-                    help="another design beside the Llama decoder of equal size (tosevik and fipitar: beside the Sufopel decoder): "
+    ap.add_argument("--design", default="", choices=("", "luzosun", "sufopel", "tosevik", "fipitar", "pobelorn"),
+                    help="another design beside the Llama decoder of equal size (tosevik and fipitar: beside the Sufopel decoder, "
+                    "pobelorn: beside the Tosevik decoder): "
                     "prefill, decode, single kernels")
     ap.add_argument("--size", default="8b", choices=tuple(DESIGN_SIZES), help="--design: the layer sizes")
     ap.add_argument("--workload-warm", type=int, default=1, help="workloads: run the workload once untimed first")

@@ -70,6 +70,59 @@ __global__ void gated_rms_kernel(const float* __restrict__ o, const T* __restric
     }
 }
 
+// four neighbouring values of a gate row, as floats
+__device__ __forceinline__ void dr_load4(const float* p, float (&x)[4]) {
+    const float4 w = *reinterpret_cast<const float4*>(p);
+    x[0] = w.x; x[1] = w.y; x[2] = w.z; x[3] = w.w;
+}
+__device__ __forceinline__ void dr_load4(const bf16* p, float (&x)[4]) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    x[0] = __uint_as_float(w.x << 16); x[1] = __uint_as_float(w.x & 0xffff0000u);
+    x[2] = __uint_as_float(w.y << 16); x[3] = __uint_as_float(w.y & 0xffff0000u);
+}
+__device__ __forceinline__ void dr_store4(float* p, const float (&x)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+}
+__device__ __forceinline__ void dr_store4(bf16* p, const float (&x)[4]) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]));
+}
+
+// The same for wide heads (a norm over all heads at once is one of them): every value is read once, kept in registers in
+// groups of four, PER groups a thread.  Everything a thread reads is sent for before the sum of squares is met.
+template <typename T, int PER>
+__global__ void __launch_bounds__(1024) gated_rms_wide_kernel(const float* __restrict__ o, const T* __restrict__ gate,
+                                                              int gate_stride, int gate_off, const float* __restrict__ w,
+                                                              T* __restrict__ out, int H, int vdim, float eps, int silu) {
+    __shared__ float scratch[32];
+    const int n = blockIdx.x, h = blockIdx.y;
+    const size_t base = ((size_t)n * H + h) * vdim;
+    const T* gp = gate + (size_t)n * gate_stride + gate_off + (size_t)h * vdim;
+    float x[PER][4], z[PER][4], wt[PER][4];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+        const int c = (i * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+        for (int e = 0; e < 4; e++) { x[i][e] = z[i][e] = 0.0f; wt[i][e] = 1.0f; }
+        if (c < vdim) {
+            dr_load4(o + base + c, x[i]);
+            dr_load4(gp + c, z[i]);
+            if (w) dr_load4(w + c, wt[i]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; e++) ss = fmaf(x[i][e], x[i][e], ss);
+    }
+    ss = mb_block_sum(ss, scratch);
+    const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
+#pragma unroll
+    for (int i = 0; i < PER; i++) {
+        const int c = (i * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+        for (int e = 0; e < 4; e++) x[i][e] = x[i][e] * r * wt[i][e] * (silu ? dr_silu(z[i][e]) : dr_sigmoid(z[i][e]));
+        if (c < vdim) dr_store4(out + base + c, x[i]);
+    }
+}
+
 template <typename T>
 static int delta_gates_launch(const T* qkv, const T* low, int low_stride, const T* wide, const float* A_log,
                               const float* dt_bias, float* q, float* k, float* v, float* g, float* beta, int N, int H, int G,
@@ -133,6 +186,15 @@ static int gated_rms_launch(const float* o, const T* gate, int gate_stride, int 
                             int H, int vdim, float eps, int silu, cudaStream_t st) {
     if (N == 0) return 0;
     if (H < 1 || H > 65535 || vdim < 1) return -2;
+    const uintptr_t ptrs = (uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out;
+    if (vdim > 256 && vdim <= 16384 && vdim % 4 == 0 && gate_stride % 4 == 0 && gate_off % 4 == 0 && (ptrs & 15) == 0) {
+        const int quads = vdim / 4, threads = quads >= 1024 ? 1024 : (quads + 31) / 32 * 32;
+#define DR_WIDE(PER) gated_rms_wide_kernel<T, PER><<<dim3(N, H), threads, 0, st>>>(o, gate, gate_stride, gate_off, w, out, H, vdim, eps, silu)
+        if (quads <= 1024) DR_WIDE(1); else if (quads <= 2048) DR_WIDE(2); else DR_WIDE(4);
+#undef DR_WIDE
+        MB_LAUNCH_CHECK();
+        return 0;
+    }
     gated_rms_kernel<T><<<dim3(N, H), vdim > 64 ? 128 : vdim > 32 ? 64 : 32, 0, st>>>(o, gate, gate_stride, gate_off, w, out,
                                                                                      H, vdim, eps, silu);
     MB_LAUNCH_CHECK();

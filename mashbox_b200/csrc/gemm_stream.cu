@@ -24,7 +24,8 @@
 //
 // Forms (EPI): 0 bf16 out; 1 SwiGLU (W = [gate rows | up rows], out = silu(gate) * up); 2 float out; 3 the float32
 // residual stream is added to in place (+ bias), and on request the product leaves what the norm after it needs: the
-// sums of squares of the new rows by 32 columns and the new rows times that norm's weight, in bf16.  (Rotation and the
+// sums of squares of the new rows by 32 columns and the new rows times that norm's weight, in bf16; 4 bf16 out, the
+// square of the product's positive part.  (Rotation and the
 // cache write stay a kernel of their own after the q/k/v product: as an epilogue here, sixteen values per thread on
 // the few warps that finish a tile, they cost 9 to 15 us against its 3.)  SCALED: the input is such a pair (rows
 // times the norm's weight in bf16, sums of squares): the token's 1/rms, computed in float from the sums, scales the
@@ -324,6 +325,10 @@ __global__ void __launch_bounds__(S_THREADS, 1) gemm_stream_kernel(const __grid_
                             if (SCALED) up *= inv_rms[n];
                             const float gt = bf16_round(v);
                             reinterpret_cast<bf16*>(out)[(size_t)n * M + m] = __float2bfloat16_rn((gt / (1.0f + expf(-gt))) * bf16_round(up));
+                        } else if (EPI == 4) {
+                            // through bf16 as when the activation is a kernel of its own
+                            const float z = fmaxf(bf16_round(v), 0.0f);
+                            reinterpret_cast<bf16*>(out)[(size_t)n * M + m] = __float2bfloat16_rn(z * z);
                         } else {
                             reinterpret_cast<bf16*>(out)[(size_t)n * M + m] = __float2bfloat16_rn(v);
                         }
@@ -496,7 +501,7 @@ static int stream_launch(const void* act, const void* W, void* out, int N, int M
     }
 }
 
-// mode 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out (N, M).
+// mode 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out (N, M); 4: bf16 out, squared ReLU.
 // ssq (or null): act holds rows of a residual stream times a norm's weight and ssq ([ceil(K / 32)][16]) the sums of
 // squares of those rows by 32 columns, as mb_gemm_stream_residual leaves them: out is then the product of
 // rmsnorm(x; weight, eps).
@@ -513,6 +518,7 @@ MB_API int mb_gemm_stream(const void* act, const float* ssq, float eps, const vo
         case 0: return stream_launch<0, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
         case 1: return stream_launch<1, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
         case 2: return stream_launch<2, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
+        case 4: return stream_launch<4, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
     }
     return -2;
 }

@@ -68,8 +68,16 @@ __device__ __forceinline__ void gv_load8_stream(const float* p, float (&v)[8]) {
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
+// a product on its way to bf16: as it is, or (MODE 5) the square of its positive part, through bf16 as when the activation
+// is a kernel of its own
+template <int MODE> __device__ __forceinline__ bf16 gv_bf16(float v) {
+    if (MODE != 5) return __float2bfloat16_rn(v);
+    const float z = fmaxf(__bfloat162float(__float2bfloat16_rn(v)), 0.0f);
+    return __float2bfloat16_rn(z * z);
+}
+
 // NT tokens (1..4).  MODE 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out; 3: out is
-// the float32 residual stream (N, M), added to.
+// the float32 residual stream (N, M), added to; 5: bf16 out (N, M), squared ReLU.
 template <int NT, int MODE, int PRE>
 __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W,
                                                              void* __restrict__ out, int M, int K, GemvNorm nrm,
@@ -259,7 +267,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const bf16* __restr
                     *xo = old[r][n] + (acc[r][n] + (bias ? bias[m0 + r] : 0.0f));
                 }
                 else if (MODE == 2) reinterpret_cast<float*>(out)[(size_t)n * M + m0 + r] = acc[r][n];
-                else reinterpret_cast<bf16*>(out)[(size_t)n * M + m0 + r] = __float2bfloat16_rn(acc[r][n]);
+                else reinterpret_cast<bf16*>(out)[(size_t)n * M + m0 + r] = gv_bf16<MODE>(acc[r][n]);
             }
         }
     }
@@ -345,7 +353,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_long_kernel(const bf16* __
             *xo = old + (s + (bias ? bias[m0 + r] : 0.0f));
         }
         else if (MODE == 2) reinterpret_cast<float*>(out)[(size_t)n * M + m0 + r] = s;
-        else reinterpret_cast<bf16*>(out)[(size_t)n * M + m0 + r] = __float2bfloat16_rn(s);
+        else reinterpret_cast<bf16*>(out)[(size_t)n * M + m0 + r] = gv_bf16<MODE>(s);
     }
 }
 
@@ -414,6 +422,9 @@ MB_API int mb_gemv_swiglu_bf16(const void* act, const void* W, void* out, int N,
 }
 MB_API int mb_gemv_f32out(const void* act, const void* W, void* out, int N, int M, int K, cudaStream_t st) {
     return gemv_launch<2, false>(act, W, out, N, M, K, GemvNorm{nullptr, nullptr, 0.0f}, nullptr, st);
+}
+MB_API int mb_gemv_relu2_bf16(const void* act, const void* W, void* out, int N, int M, int K, cudaStream_t st) {
+    return gemv_launch<5, false>(act, W, out, N, M, K, GemvNorm{nullptr, nullptr, 0.0f}, nullptr, st);
 }
 // x (N, M) float32 += act W^T + bias (bias may be null)
 MB_API int mb_gemv_residual(const void* act, const void* W, float* x, const float* bias, int N, int M, int K, cudaStream_t st) {

@@ -918,10 +918,12 @@ def linear_gemv_residual(a, w, x, bias=None):
 
 
 def linear_gemv(a, w, out, mode="plain"):
-    """a (N <= 4, K) bf16, w (M, K) bf16 ("swiglu": (2M, K)) -> out (N, M): bf16, or float32 for mode "float"."""
+    """a (N <= 4, K) bf16, w (M, K) bf16 ("swiglu": (2M, K)) -> out (N, M): bf16 ("relu2": squared ReLU of the product), or
+    float32 for mode "float"."""
     _cuda(a, w, out)
     N, K = a.shape
-    name = {"plain": "mb_gemv_bf16", "swiglu": "mb_gemv_swiglu_bf16", "float": "mb_gemv_f32out"}[mode]
+    name = {"plain": "mb_gemv_bf16", "swiglu": "mb_gemv_swiglu_bf16", "float": "mb_gemv_f32out",
+            "relu2": "mb_gemv_relu2_bf16"}[mode]
     f = _fn("gemv", name, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(f(_p(a), _p(w), _p(out), N, out.shape[1], K, _stream()), "gemv")
     return out
@@ -978,7 +980,8 @@ def _stream_buffers(device, M):
 
 
 def linear_stream(a, w, out, mode="plain", sums=None, eps=0.0):
-    """a (N <= 16, K) bf16, w (M, K) bf16 ("swiglu": (2M, K)) -> out (N, M): bf16, or float32 for mode "float".
+    """a (N <= 16, K) bf16, w (M, K) bf16 ("swiglu": (2M, K)) -> out (N, M): bf16 ("relu2": squared ReLU of the product), or
+    float32 for mode "float".
     sums (ceil(K / 32), 16) float32, if given: a holds rows of a residual stream times a norm's weight and sums the sums
     of squares of those rows by 32 columns, as linear_stream_residual leaves them; out is then the product of
     rmsnorm(x; weight, eps): 1 / rms scales the float sums of the product."""
@@ -988,7 +991,7 @@ def linear_stream(a, w, out, mode="plain", sums=None, eps=0.0):
     ws, cnt = _stream_buffers(a.device, M)
     f = _fn("gemm_stream", "mb_gemm_stream", [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                               c_void_p, c_void_p, c_void_p, c_void_p])
-    _check(f(_p(a), _p(sums), float(eps), _p(w), _p(out), N, M, K, {"plain": 0, "swiglu": 1, "float": 2}[mode], _p(ws),
+    _check(f(_p(a), _p(sums), float(eps), _p(w), _p(out), N, M, K, {"plain": 0, "swiglu": 1, "float": 2, "relu2": 4}[mode], _p(ws),
              _p(cnt), _p(error_word(a.device)), _stream()), "gemm_stream")
     return out
 
@@ -1075,8 +1078,10 @@ def linear_xielu(a, w, out, ap, an):
 
 
 def fused_relu2_supports(N, F, K, dtype):
-    """the up product of a bfloat16 prompt portion with the squared ReLU in its epilogue (the tcgen05 product)"""
-    return dtype == torch.bfloat16 and tc5_supports(N, F, K, "swiglu")
+    """the up product with the squared ReLU in its epilogue: the tcgen05 product for prompt portions, the matrix-vector or
+    the weight-streaming kernel for decode batches (bfloat16)"""
+    return dtype == torch.bfloat16 and F % 8 == 0 and (gemv_supports(N, K) or stream_supports(N, K)
+                                                       or tc5_supports(N, F, K, "swiglu"))
 
 
 def linear_relu2(a, w, out):
@@ -1086,6 +1091,10 @@ def linear_relu2(a, w, out):
     if not (fused_relu2_supports(N, out.shape[1], K, a.dtype) and a.is_contiguous() and w.is_contiguous()
             and out.is_contiguous()):
         raise KernelError("linear_relu2: no fused kernel takes these sizes")
+    if gemv_supports(N, K):
+        return linear_gemv(a, w, out, "relu2")
+    if stream_supports(N, K):
+        return linear_stream(a, w, out, "relu2")
     f = _fn("gemm_tc5", "mb_gemm_tc5_relu2_bf16", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(f(_p(a), _p(w), _p(out), N, out.shape[1], K, _p(error_word(a.device)), _stream()), "gemm_tc5_relu2")
     return out

@@ -338,12 +338,16 @@ def test_squared_relu_alone_and_in_the_products_epilogue(dtype):
         ops.relu2(dev(z, dtype), out)
         kernel_close(out, torch.clamp(z, min=0) ** 2, dtype, "max(z, 0)^2", 1e-2 if dtype == "bfloat16" else None)
     if dtype == "bfloat16":
-        for N, F, K in ((128, 256, 64), (200, 264, 328), (515, 1032, 128)):
+        # one token (matrix-vector, short and long rows), a decode batch (weight-streaming), prompt portions (tcgen05)
+        ops.configure({})
+        for N, F, K in ((1, 264, 64), (1, 72, 8448), (1, 40, 2568), (2, 96, 1024), (5, 136, 4096), (16, 4104, 328), (9, 24, 72),
+                        (128, 256, 64), (200, 264, 328), (515, 1032, 128)):
             a, w = rnd(gen, N, K, dtype=dtype), rnd(gen, F, K, dtype=dtype, scale=K ** -0.5)
             out = torch.full((N, F), float("nan"), device=DEV, dtype=torch.bfloat16)
             assert ops.fused_relu2_supports(N, F, K, torch.bfloat16)
             ops.linear_relu2(dev(a, dtype), dev(w, dtype), out)
             kernel_close(out, torch.clamp(a @ w.T, min=0) ** 2, dtype, f"product {N} x {F} x {K}")
+        assert not ops.fused_relu2_supports(64, 256, 64, torch.bfloat16) and not ops.fused_relu2_supports(5, 100, 64, torch.bfloat16)
 
 
 # ------------------------------------------------------------------------------------------------ the model in the engine

@@ -53,13 +53,17 @@ def _builtin():
     if _done:
         return
     _done = True
-    from ..models import fipitar, llama, luzosun, pobelorn, sufopel, tosevik
+    from ..models import fipitar, llama, lorozen, luzosun, pobelorn, sufopel, tosevik
     from .fipitar import FipitarConfig
     from .llama import LlamaConfig
+    from .lorozen import LorozenConfig
     from .luzosun import LuzosunConfig
     from .pobelorn import PobelornConfig
     from .sufopel import SufopelConfig
     from .tosevik import TosevikConfig
+    if "Lorozen" not in ARCHITECTURES:
+        register_architecture(Architecture("Lorozen", LorozenConfig, lorozen.model_spec, lorozen.canonical_names,
+                                           lorozen.stored_tensors))
     if "Pobelorn" not in ARCHITECTURES:
         register_architecture(Architecture("Pobelorn", PobelornConfig, pobelorn.model_spec, pobelorn.canonical_names,
                                            pobelorn.stored_tensors))

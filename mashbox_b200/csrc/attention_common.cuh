@@ -15,6 +15,7 @@ struct AttnParams {
     int* counters;                          // one per (first item of a split group, kv head), zero between launches; or null
     int H, KV, G, page, num_pages, window;
     int keep = 0;                           // behind the window the first `keep` positions stay visible (0 without a window)
+    const float* sinks = nullptr;           // per query head: a score that joins the softmax's denominator without a value, or null
     int page_shift;                         // log2(page) when the page size is a power of two, else -1
     float scale_log2;
     int* err;

@@ -424,6 +424,9 @@ __global__ void __launch_bounds__(T5_THREADS, 1) attn_tc5_kernel(const AttnParam
             }
 #ifndef T5_SIG
             float m_run = -INFINITY, l_run = 0.0f;
+#ifndef T5_DIFF
+            if (P.sinks && r < R) { m_run = P.sinks[kvh * G + r % G] * 1.4426950408889634f; l_run = 1.0f; }    // a key without a value
+#endif
 #else
             // the row's head: slope and bias in units of log2 e, as the exponent of 2^x wants them
             const int hq = kvh * G + (r < R ? r % G : 0);
@@ -748,6 +751,7 @@ MB_API int T5_ENTRY(const void* q, int q_stride, void* out, const void* kpool, c
 #endif
 #if !defined(T5_DIFF) && !defined(T5_SIG)
                             int keep,                                           // first positions seen behind the window
+                            const float* sinks,                                 // per query head, or null
 #endif
                             int* err, cudaStream_t st) {
     if (n_items == 0) return 0;
@@ -768,6 +772,7 @@ MB_API int T5_ENTRY(const void* q, int q_stride, void* out, const void* kpool, c
     P.H = H; P.KV = KV; P.G = H / KV; P.page = page; P.num_pages = num_pages; P.window = window;
 #if !defined(T5_DIFF) && !defined(T5_SIG)
     P.keep = window > 0 ? keep : 0;
+    P.sinks = sinks;
 #endif
     P.page_shift = -1;
     for (int sft = 0; sft < 31; sft++) if ((1 << sft) == page) P.page_shift = sft;

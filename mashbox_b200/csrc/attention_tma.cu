@@ -206,6 +206,18 @@ __global__ void __launch_bounds__(160, 2) attn_tma_kernel(const AttnParams P, co
         }
     }
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
+    if (P.sinks && split == 0 && (!DECODE || warp == 0)) {
+        // a sink: the row starts with that score as its maximum and a sum of one (in the sum of one of its four threads,
+        // of one of the warps and splits that share the row), and an empty output
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int r = row0 + m0 + g + i * 8;
+            if (r < R) {
+                m_run[i] = P.sinks[kvh * G + r % G] * 1.4426950408889634f;
+                l_run[i] = tig == 0 ? 1.0f : 0.0f;
+            }
+        }
+    }
     float o[DT][4];
 #pragma unroll
     for (int d = 0; d < DT; d++) { o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.0f; }
@@ -628,7 +640,7 @@ static int attn_tma_run(const void* q, int q_stride, void* out, const void* kpoo
                         const int* pos0, const int* part_base, const int* seq_row, const int* table, int max_blocks,
                         float* part_o, float* part_ml, int max_splits, int H, int KV, int HD, int page, int num_pages,
                         int window, float scale, int* counters, int* err, cudaStream_t st, int fuse, const float* bias,
-                        const float* freqs, int RD, int pairing, int cluster = 0, int keep = 0) {
+                        const float* freqs, int RD, int pairing, int cluster = 0, int keep = 0, const float* sinks = nullptr) {
     if (n_items == 0) return 0;
     if (cluster > 1 && (!decode || cluster > 8)) return -2;
     if (!mb_attn_tma_supports(HD, page) || KV < 1 || H % KV || KV > 65535) return -2;
@@ -642,6 +654,7 @@ static int attn_tma_run(const void* q, int q_stride, void* out, const void* kpoo
     P.part_o = part_o; P.part_ml = part_ml; P.max_splits = max_splits; P.counters = counters;
     P.H = H; P.KV = KV; P.G = H / KV; P.page = page; P.num_pages = num_pages; P.window = window;
     P.keep = window > 0 ? keep : 0;
+    P.sinks = sinks;
     P.page_shift = -1;
     for (int sft = 0; sft < 31; sft++) if ((1 << sft) == page) P.page_shift = sft;
     P.scale_log2 = scale * 1.4426950408889634f;
@@ -666,10 +679,10 @@ MB_API int mb_attn_tma_bf16(const void* q, int q_stride, void* out, const void* 
                             const void* items, int n_items, int decode, const int* q_start, const int* q_len,
                             const int* pos0, const int* part_base, const int* seq_row, const int* table, int max_blocks,
                             float* part_o, float* part_ml, int max_splits, int H, int KV, int HD, int page, int num_pages,
-                            int window, int keep, float scale, int* counters, int* err, cudaStream_t st) {
+                            int window, int keep, const float* sinks, float scale, int* counters, int* err, cudaStream_t st) {
     return attn_tma_run(q, q_stride, out, kpool, vpool, items, n_items, decode, q_start, q_len, pos0, part_base, seq_row,
                         table, max_blocks, part_o, part_ml, max_splits, H, KV, HD, page, num_pages, window, scale,
-                        counters, err, st, 0, nullptr, nullptr, 0, 0, 0, keep);
+                        counters, err, st, 0, nullptr, nullptr, 0, 0, 0, keep, sinks);
 }
 
 // The decode form for a step in which every sequence brings one token, with the rotate-and-store step folded in: qkv
@@ -678,12 +691,12 @@ MB_API int mb_attn_tma_bf16(const void* q, int q_stride, void* out, const void* 
 MB_API int mb_attn_tma_rope_bf16(const void* qkv, int q_stride, void* out, void* kpool, void* vpool, const void* items,
                                  int n_items, const int* q_start, const int* q_len, const int* pos0, const int* part_base,
                                  const int* seq_row, const int* table, int max_blocks, float* part_o, float* part_ml,
-                                 int max_splits, int H, int KV, int HD, int page, int num_pages, int window, int keep, float scale,
+                                 int max_splits, int H, int KV, int HD, int page, int num_pages, int window, int keep, const float* sinks, float scale,
                                  int* counters, int* err, const float* bias, const float* freqs, int RD, int pairing,
                                  cudaStream_t st) {
     return attn_tma_run(qkv, q_stride, out, kpool, vpool, items, n_items, 1, q_start, q_len, pos0, part_base, seq_row, table,
                         max_blocks, part_o, part_ml, max_splits, H, KV, HD, page, num_pages, window, scale, counters,
-                        err, st, 1, bias, freqs, RD, pairing, 0, keep);
+                        err, st, 1, bias, freqs, RD, pairing, 0, keep, sinks);
 }
 
 // The decode form launched as thread-block clusters: every sequence of the launch is cut into `cluster` splits (2 to
@@ -693,12 +706,12 @@ MB_API int mb_attn_tma_rope_bf16(const void* qkv, int q_stride, void* out, void*
 MB_API int mb_attn_tma_cluster_bf16(const void* q, int q_stride, void* out, void* kpool, void* vpool, const void* items,
                                     int n_items, const int* q_start, const int* q_len, const int* pos0, const int* seq_row,
                                     const int* table, int max_blocks, int cluster, int H, int KV, int HD, int page,
-                                    int num_pages, int window, int keep, float scale, int* err, int rope, const float* bias,
+                                    int num_pages, int window, int keep, const float* sinks, float scale, int* err, int rope, const float* bias,
                                     const float* freqs, int RD, int pairing, cudaStream_t st) {
     if (cluster < 2) return -2;
     return attn_tma_run(q, q_stride, out, kpool, vpool, items, n_items, 1, q_start, q_len, pos0, nullptr, seq_row, table,
                         max_blocks, nullptr, nullptr, cluster, H, KV, HD, page, num_pages, window, scale, nullptr, err, st,
-                        rope, bias, freqs, RD, pairing, cluster, keep);
+                        rope, bias, freqs, RD, pairing, cluster, keep, sinks);
 }
 
 static int attn_tma_query(int HD, int rope, int what) {

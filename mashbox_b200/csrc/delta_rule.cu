@@ -13,8 +13,8 @@
 //   delta_gates   from the (convolved) q/k/v product and the small products: silu; q and k to unit vectors per head (q
 //                 also times dim^-1/2); beta = sigmoid; g = exp(-exp(A) softplus(a + dt_bias)); all left in float32
 //   delta_rule    the recurrence
-//   gated_rms     o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) per head, to the storage type (w may be absent; the gate
-//                 may be silu(gate) instead)
+//   gated_rms     o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) per head, to the storage type (w may be absent, one for all heads
+//                 or, w_head values apart, one per head; the gate may be silu(gate) instead)
 #include "common.cuh"
 
 #include "linear_scan.cuh"
@@ -55,7 +55,7 @@ __global__ void delta_gates_kernel(const T* __restrict__ qkv, const T* __restric
 // grid (N, H): o (N, H vdim) float32 -> out in the storage type
 template <typename T>
 __global__ void gated_rms_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_stride, int gate_off,
-                                 const float* __restrict__ w, T* __restrict__ out, int H, int vdim, float eps, int silu) {
+                                 const float* __restrict__ w, T* __restrict__ out, int H, int vdim, float eps, int silu, int w_head) {
     __shared__ float scratch[32];
     const int n = blockIdx.x, h = blockIdx.y;
     const float* src = o + ((size_t)n * H + h) * vdim;
@@ -66,7 +66,7 @@ __global__ void gated_rms_kernel(const float* __restrict__ o, const T* __restric
     const T* gp = gate + (size_t)n * gate_stride + gate_off + (size_t)h * vdim;
     for (int c = threadIdx.x; c < vdim; c += blockDim.x) {
         const float z = mb_load(gp + c);
-        mb_store(out + ((size_t)n * H + h) * vdim + c, src[c] * r * (w ? w[c] : 1.0f) * (silu ? dr_silu(z) : dr_sigmoid(z)));
+        mb_store(out + ((size_t)n * H + h) * vdim + c, src[c] * r * (w ? w[(size_t)h * w_head + c] : 1.0f) * (silu ? dr_silu(z) : dr_sigmoid(z)));
     }
 }
 
@@ -92,7 +92,7 @@ __device__ __forceinline__ void dr_store4(bf16* p, const float (&x)[4]) {
 template <typename T, int PER>
 __global__ void __launch_bounds__(1024) gated_rms_wide_kernel(const float* __restrict__ o, const T* __restrict__ gate,
                                                               int gate_stride, int gate_off, const float* __restrict__ w,
-                                                              T* __restrict__ out, int H, int vdim, float eps, int silu) {
+                                                              T* __restrict__ out, int H, int vdim, float eps, int silu, int w_head) {
     __shared__ float scratch[32];
     const int n = blockIdx.x, h = blockIdx.y;
     const size_t base = ((size_t)n * H + h) * vdim;
@@ -107,7 +107,7 @@ __global__ void __launch_bounds__(1024) gated_rms_wide_kernel(const float* __res
         if (c < vdim) {
             dr_load4(o + base + c, x[i]);
             dr_load4(gp + c, z[i]);
-            if (w) dr_load4(w + c, wt[i]);
+            if (w) dr_load4(w + (size_t)h * w_head + c, wt[i]);
         }
 #pragma unroll
         for (int e = 0; e < 4; e++) ss = fmaf(x[i][e], x[i][e], ss);
@@ -183,30 +183,30 @@ MB_API int mb_delta_rule(const float* q, const float* k, const float* v, const f
 
 template <typename T>
 static int gated_rms_launch(const float* o, const T* gate, int gate_stride, int gate_off, const float* w, T* out, int N,
-                            int H, int vdim, float eps, int silu, cudaStream_t st) {
+                            int H, int vdim, float eps, int silu, int w_head, cudaStream_t st) {
     if (N == 0) return 0;
     if (H < 1 || H > 65535 || vdim < 1) return -2;
     const uintptr_t ptrs = (uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out;
-    if (vdim > 256 && vdim <= 16384 && vdim % 4 == 0 && gate_stride % 4 == 0 && gate_off % 4 == 0 && (ptrs & 15) == 0) {
+    if (vdim > 256 && vdim <= 16384 && vdim % 4 == 0 && gate_stride % 4 == 0 && gate_off % 4 == 0 && w_head % 4 == 0 && (ptrs & 15) == 0) {
         const int quads = vdim / 4, threads = quads >= 1024 ? 1024 : (quads + 31) / 32 * 32;
-#define DR_WIDE(PER) gated_rms_wide_kernel<T, PER><<<dim3(N, H), threads, 0, st>>>(o, gate, gate_stride, gate_off, w, out, H, vdim, eps, silu)
+#define DR_WIDE(PER) gated_rms_wide_kernel<T, PER><<<dim3(N, H), threads, 0, st>>>(o, gate, gate_stride, gate_off, w, out, H, vdim, eps, silu, w_head)
         if (quads <= 1024) DR_WIDE(1); else if (quads <= 2048) DR_WIDE(2); else DR_WIDE(4);
 #undef DR_WIDE
         MB_LAUNCH_CHECK();
         return 0;
     }
     gated_rms_kernel<T><<<dim3(N, H), vdim > 64 ? 128 : vdim > 32 ? 64 : 32, 0, st>>>(o, gate, gate_stride, gate_off, w, out,
-                                                                                     H, vdim, eps, silu);
+                                                                                     H, vdim, eps, silu, w_head);
     MB_LAUNCH_CHECK();
     return 0;
 }
 
 MB_API int mb_gated_rms_f32(const float* o, const void* gate, int gate_stride, int gate_off, const float* w, void* out, int N,
-                            int H, int vdim, float eps, int silu, cudaStream_t st) {
-    return gated_rms_launch<float>(o, (const float*)gate, gate_stride, gate_off, w, (float*)out, N, H, vdim, eps, silu, st);
+                            int H, int vdim, float eps, int silu, int w_head, cudaStream_t st) {
+    return gated_rms_launch<float>(o, (const float*)gate, gate_stride, gate_off, w, (float*)out, N, H, vdim, eps, silu, w_head, st);
 }
 
 MB_API int mb_gated_rms_bf16(const float* o, const void* gate, int gate_stride, int gate_off, const float* w, void* out, int N,
-                             int H, int vdim, float eps, int silu, cudaStream_t st) {
-    return gated_rms_launch<bf16>(o, (const bf16*)gate, gate_stride, gate_off, w, (bf16*)out, N, H, vdim, eps, silu, st);
+                             int H, int vdim, float eps, int silu, int w_head, cudaStream_t st) {
+    return gated_rms_launch<bf16>(o, (const bf16*)gate, gate_stride, gate_off, w, (bf16*)out, N, H, vdim, eps, silu, w_head, st);
 }

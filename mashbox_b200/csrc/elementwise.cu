@@ -497,18 +497,23 @@ MB_API int mb_patch_tokens(int* dst, const int* src, const int* pairs, int n, cu
 
 // ------------------------------------------------------------------------------------------------ SwiGLU
 // gu[n] = [gate (F) | up (F)] -> out[n, f] = silu(gate) * up
-template <typename T>
+// the gate of a gated unit: silu, or the tanh form of gelu
+template <bool GELU> __device__ __forceinline__ float glu_gate(float g) {
+    return GELU ? mb_gelu_tanh(g) : g / (1.0f + expf(-g));
+}
+
+template <typename T, bool GELU>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, size_t total) {
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     const size_t n = i / F, f = i % F;
     const float g = mb_load(gu + n * 2 * F + f), u = mb_load(gu + n * 2 * F + F + f);
-    mb_store(out + i, (g / (1.0f + expf(-g))) * u);
+    mb_store(out + i, glu_gate<GELU>(g) * u);
 }
 
 
 // the same, eight values per thread, for F a multiple of 8: block (x: chunks of a row), grid.y: rows
-template <typename T>
+template <typename T, bool GELU>
 __global__ void swiglu_vec_kernel(const T* __restrict__ gu, T* __restrict__ out, int F) {
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= F / 8) return;
@@ -517,7 +522,7 @@ __global__ void swiglu_vec_kernel(const T* __restrict__ gu, T* __restrict__ out,
     load8(gu + n * 2 * F + c * 8, g);
     load8(gu + n * 2 * F + F + c * 8, u);
 #pragma unroll
-    for (int e = 0; e < 8; e++) g[e] = (g[e] / (1.0f + expf(-g[e]))) * u[e];
+    for (int e = 0; e < 8; e++) g[e] = glu_gate<GELU>(g[e]) * u[e];
     store8(out + n * F + c * 8, g);
 }
 
@@ -680,22 +685,29 @@ MB_API int mb_rope_kv_write_bf16(void* qkv, const float* bias, const int* positi
                                                N, H, KV, HD, RD, pairing, page, num_pages, err, st);
 }
 
-template <typename T>
+template <typename T, bool GELU>
 static int swiglu_launch(const void* gu, void* out, int N, int F, cudaStream_t st) {
     const size_t total = (size_t)N * F;
     if (total == 0) return 0;
     if (F % 8 == 0 && N <= 65535)
-        swiglu_vec_kernel<T><<<dim3((F / 8 + 127) / 128, N), 128, 0, st>>>((const T*)gu, (T*)out, F);
+        swiglu_vec_kernel<T, GELU><<<dim3((F / 8 + 127) / 128, N), 128, 0, st>>>((const T*)gu, (T*)out, F);
     else
-        swiglu_kernel<T><<<(unsigned)((total + 255) / 256), 256, 0, st>>>((const T*)gu, (T*)out, F, total);
+        swiglu_kernel<T, GELU><<<(unsigned)((total + 255) / 256), 256, 0, st>>>((const T*)gu, (T*)out, F, total);
     MB_LAUNCH_CHECK();
     return 0;
 }
 MB_API int mb_swiglu_f32(const void* gu, void* out, int N, int F, cudaStream_t st) {
-    return swiglu_launch<float>(gu, out, N, F, st);
+    return swiglu_launch<float, false>(gu, out, N, F, st);
 }
 MB_API int mb_swiglu_bf16(const void* gu, void* out, int N, int F, cudaStream_t st) {
-    return swiglu_launch<__nv_bfloat16>(gu, out, N, F, st);
+    return swiglu_launch<__nv_bfloat16, false>(gu, out, N, F, st);
+}
+// the same with the tanh form of gelu on the gate
+MB_API int mb_geglu_f32(const void* gu, void* out, int N, int F, cudaStream_t st) {
+    return swiglu_launch<float, true>(gu, out, N, F, st);
+}
+MB_API int mb_geglu_bf16(const void* gu, void* out, int N, int F, cudaStream_t st) {
+    return swiglu_launch<__nv_bfloat16, true>(gu, out, N, F, st);
 }
 
 // ------------------------------------------------------------------------------------------------ clamped gated unit

@@ -8,7 +8,7 @@
 //                 decay = exp(-exp(A_log) dt)
 //     ssd_out     y = o + D x;  y <- y silu(z);  each of `parts` equal stretches of a row divided by its own root mean
 //                 square;  times a weight;  to the storage type
-//   gated_scan    the recurrence itself (the kernel template shared with the delta rule; modes 1 and 2)
+//   gated_scan    the recurrence itself (the kernel template shared with the delta rule; modes 1, 2 and 3)
 //
 // Decays, their logarithms, softplus, dt, the state and the recurrence are float32 whatever the storage type.
 #include "linear_scan.cuh"
@@ -112,12 +112,13 @@ __global__ void ssd_out_kernel(const float* __restrict__ o, const T* __restrict_
 GS_ENTRIES(f32, float)
 GS_ENTRIES(bf16, bf16)
 
-// per_head 0: g (N, H, dim); 1: g (N, H).  state (slots, ..): head h's matrix (dim, vdim) at h dim vdim.
-MB_API int mb_gated_scan(const float* q, const float* k, const float* v, const float* g, float* o, float* state,
+// per_head 0: g (N, H, dim); 1: g (N, H).  beta (N, H) (or null; with per_head 0): the read-out comes before the token joins
+// the state, plus beta times the token's value.  state (slots, ..): head h's matrix (dim, vdim) at h dim vdim.
+MB_API int mb_gated_scan(const float* q, const float* k, const float* v, const float* g, const float* beta, float* o, float* state,
                          long long state_stride, const int* q_start, const int* q_len, const int* state_slot, int S, int H,
                          int G, int dim, int vdim, int per_head, int long_stretches, cudaStream_t st) {
     if (S == 0) return 0;
-    if (G < 1 || H % G || H > 65535 || S > 65535 || dim < 1 || dim > 256 || vdim < 1) return -2;
+    if (G < 1 || H % G || H > 65535 || S > 65535 || dim < 1 || dim > 256 || vdim < 1 || (beta && per_head)) return -2;
 #define GS_LAUNCH(LANES, R4, MODE)                                                                                         \
     {                                                                                                                      \
         const int cols = DR_THREADS / LANES * DR_CPT;                                                                      \
@@ -130,13 +131,13 @@ MB_API int mb_gated_scan(const float* q, const float* k, const float* v, const f
             configured = true;                                                                                             \
         }                                                                                                                  \
         delta_rule_kernel<LANES, R4, MODE><<<dim3((vdim + cols - 1) / cols, H, S), DR_THREADS, smem, st>>>(                \
-            q, k, v, g, nullptr, o, state, state_stride, q_start, q_len, state_slot, H, G, dim, vdim);                     \
+            q, k, v, g, beta, o, state, state_stride, q_start, q_len, state_slot, H, G, dim, vdim);                     \
         MB_LAUNCH_CHECK();                                                                                                 \
         return 0;                                                                                                          \
     }
 #define GS_CASE(LANES, R4)                                                                                                 \
     if (dim <= 4 * R4 * LANES) {                                                                                           \
-        if (per_head) GS_LAUNCH(LANES, R4, 2) else GS_LAUNCH(LANES, R4, 1)                                                 \
+        if (per_head) GS_LAUNCH(LANES, R4, 2) else if (beta) GS_LAUNCH(LANES, R4, 3) else GS_LAUNCH(LANES, R4, 1)          \
     }
     // Wide keys: more threads a column where sequences bring long stretches (a prompt gives few blocks, and the chain of one
     // token is shorter with fewer values a thread: 523 against 649 us on 2,048 tokens of 16 heads of 128 x 128), fewer where

@@ -8,7 +8,7 @@
 #define BK 16
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W,
-                                                        float* __restrict__ C, int N, int M, int K) {
+                                                        float* __restrict__ C, int N, int M, int K, int ldc) {
     __shared__ float As[BK][TILE + 4];
     __shared__ float Ws[BK][TILE + 4];
     const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;       // tx: 4 output columns (m), ty: 4 output rows (n)
@@ -50,16 +50,18 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int m = m0 + tx * 4 + j;
-            if (m < M) C[(size_t)n * M + m] = acc[i][j];
+            if (m < M) C[(size_t)n * ldc + m] = acc[i][j];
         }
     }
 }
 
-MB_API int mb_gemm_f32(const float* A, const float* W, float* C, int N, int M, int K, cudaStream_t st) {
+// rows of C are ldc floats apart
+MB_API int mb_gemm_f32(const float* A, const float* W, float* C, int N, int M, int K, int ldc, cudaStream_t st) {
     if (N == 0 || M == 0) return 0;
+    if (ldc < M) return -2;
     dim3 grid((M + TILE - 1) / TILE, (N + TILE - 1) / TILE);
     if (grid.y > 65535) return -2;
-    gemm_f32_kernel<<<grid, 256, 0, st>>>(A, W, C, N, M, K);
+    gemm_f32_kernel<<<grid, 256, 0, st>>>(A, W, C, N, M, K, ldc);
     MB_LAUNCH_CHECK();
     return 0;
 }

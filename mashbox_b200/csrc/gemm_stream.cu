@@ -25,7 +25,7 @@
 // Forms (EPI): 0 bf16 out; 1 SwiGLU (W = [gate rows | up rows], out = silu(gate) * up); 2 float out; 3 the float32
 // residual stream is added to in place (+ bias), and on request the product leaves what the norm after it needs: the
 // sums of squares of the new rows by 32 columns and the new rows times that norm's weight, in bf16; 4 bf16 out, the
-// square of the product's positive part.  (Rotation and the
+// square of the product's positive part; 5 as 1 with the tanh form of gelu.  (Rotation and the
 // cache write stay a kernel of their own after the q/k/v product: as an epilogue here, sixteen values per thread on
 // the few warps that finish a tile, they cost 9 to 15 us against its 3.)  SCALED: the input is such a pair (rows
 // times the norm's weight in bf16, sums of squares): the token's 1/rms, computed in float from the sums, scales the
@@ -100,7 +100,7 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
 
 // compile-time shape of a kernel: TH rows of W per tile (128, 64 or 32)
 template <int EPI, int TH> struct StreamShape {
-    static constexpr int SETS = EPI == 1 ? 2 : 1;
+    static constexpr int SETS = EPI == 1 || EPI == 5 ? 2 : 1;
     static constexpr int MG = TH / 32;                  // consumer warps side by side along the rows of a tile
     static constexpr int KG = 4 / MG;                   // ... and along k: warp w takes the boxes b with b % KG == w / MG
     static constexpr int NB = 2 * KG;                   // boxes of 64 k per set and stage
@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(S_THREADS, 1) gemm_stream_kernel(const __grid_
                                                                     void* __restrict__ out, int N, int M, int K, int tiles,
                                                                     float* __restrict__ partial, int* __restrict__ tile_done,
                                                                     StreamNorm nrm, const float* __restrict__ bias,
-                                                                    StreamAfter after, int* err) {
+                                                                    StreamAfter after, int* err, int group_rows) {
     using SH = StreamShape<EPI, TH>;
     constexpr int SETS = SH::SETS, MG = SH::MG, KG = SH::KG, NB = SH::NB, KS = SH::KS, BOX = SH::BOX;
     constexpr int STAGE = SH::STAGE, STAGES = SH::STAGES;
@@ -150,9 +150,9 @@ __global__ void __launch_bounds__(S_THREADS, 1) gemm_stream_kernel(const __grid_
             const int k = kb * KS + b * 64;
             if (what & 1) {
                 tma_load_2d(dst + b * BOX, &wmap, k, row, fb);
-                if (EPI == 1) tma_load_2d(dst + S_W_BYTES + b * BOX, &wmap, k, M + row, fb);
+                if (SETS == 2) tma_load_2d(dst + S_W_BYTES + b * BOX, &wmap, k, M + row, fb);
             }
-            if (what & 2) tma_load_2d(dst + SETS * S_W_BYTES + b * S_XBOX, &xmap, k, 0, fb);
+            if (what & 2) tma_load_2d(dst + SETS * S_W_BYTES + b * S_XBOX, &xmap, k, group_rows ? row / group_rows * N : 0, fb);
         }
     };
     StreamWalk pw(range);                                             // the producer's place (thread 0 only)
@@ -319,12 +319,12 @@ __global__ void __launch_bounds__(S_THREADS, 1) gemm_stream_kernel(const __grid_
                             reinterpret_cast<float*>(out)[(size_t)n * M + m] = v;
                             if (after.scaled) after.scaled[(size_t)n * M + m] = __float2bfloat16_rn(v * row_w[((a >> 3) & 1) * 2 + ((a >> 1) & 1)]);
                             accf[a] = v;
-                        } else if (EPI == 1) {
+                        } else if (EPI == 1 || EPI == 5) {
                             // gate and up pass through bf16 as they do when the products are separate kernels
                             float up = accf[(SETS - 1) * 16 + a];
                             if (SCALED) up *= inv_rms[n];
                             const float gt = bf16_round(v);
-                            reinterpret_cast<bf16*>(out)[(size_t)n * M + m] = __float2bfloat16_rn((gt / (1.0f + expf(-gt))) * bf16_round(up));
+                            reinterpret_cast<bf16*>(out)[(size_t)n * M + m] = __float2bfloat16_rn((EPI == 5 ? mb_gelu_tanh(gt) : gt / (1.0f + expf(-gt))) * bf16_round(up));
                         } else if (EPI == 4) {
                             // through bf16 as when the activation is a kernel of its own
                             const float z = fmaxf(bf16_round(v), 0.0f);
@@ -465,13 +465,13 @@ MB_PDL_SWITCH(mb_gemm_stream_set_pdl)
 
 template <int EPI, bool SCALED, int TH>
 static int stream_launch_th(const void* act, const void* W, void* out, int N, int M, int K, float* workspace, int* counters,
-                            StreamNorm nrm, const float* bias, StreamAfter after, int* err, cudaStream_t st, long long grid) {
+                            StreamNorm nrm, const float* bias, StreamAfter after, int* err, cudaStream_t st, long long grid, int groups) {
     using SH = StreamShape<EPI, TH>;
     static_assert(SH::STAGES >= 2, "a ring of at least two stages");
     CUtensorMap wmap, xmap;
     int rc = matrix_map(W, (long long)SH::SETS * M, K, TH, &wmap);
     if (rc) return rc;
-    if ((rc = matrix_map(act, N, K, S_NT, &xmap))) return rc;
+    if ((rc = matrix_map(act, (long long)groups * N, K, S_NT, &xmap))) return rc;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(gemm_stream_kernel<EPI, SCALED, TH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SH::BYTES);
@@ -482,26 +482,29 @@ static int stream_launch_th(const void* act, const void* W, void* out, int N, in
     const long long T = (long long)tiles * ((K + SH::KS - 1) / SH::KS);
     if (grid > T) grid = T;
     const cudaError_t e = mb_launch(mb_pdl != 0, gemm_stream_kernel<EPI, SCALED, TH>, dim3((unsigned)grid), dim3(S_THREADS),
-                                    SH::BYTES, st, wmap, xmap, out, N, M, K, tiles, workspace, counters, nrm, bias, after, err);
+                                    SH::BYTES, st, wmap, xmap, out, N, M, K, tiles, workspace, counters, nrm, bias, after, err,
+                                    groups > 1 ? M / groups : 0);
     return e == cudaSuccess ? 0 : (int)e;
 }
 
 template <int EPI, bool SCALED>
 static int stream_launch(const void* act, const void* W, void* out, int N, int M, int K, float* workspace, int* counters,
-                         StreamNorm nrm, const float* bias, StreamAfter after, int* err, cudaStream_t st) {
+                         StreamNorm nrm, const float* bias, StreamAfter after, int* err, cudaStream_t st, int groups = 1) {
     if (N == 0 || M == 0) return 0;
     if (N > S_NT || K % 8 || K < 8 || !workspace || !counters || (reinterpret_cast<uintptr_t>(W) & 15) ||
         (reinterpret_cast<uintptr_t>(act) & 15) || (SCALED && (!nrm.ssq || (reinterpret_cast<uintptr_t>(nrm.ssq) & 15))))
         return -2;
-    const StreamPlan plan = stream_plan(M, K, EPI == 1 ? 2 : 1, stream_sms(), 32);
+    const StreamPlan plan = stream_plan(M, K, EPI == 1 || EPI == 5 ? 2 : 1, stream_sms(), 32);
+    if (groups < 1 || (groups > 1 && M % (groups * 128))) return -2;        // a row tile reads one group's activations
     switch (plan.th) {
-        case 128: return stream_launch_th<EPI, SCALED, 128>(act, W, out, N, M, K, workspace, counters, nrm, bias, after, err, st, plan.grid);
-        case 64: return stream_launch_th<EPI, SCALED, 64>(act, W, out, N, M, K, workspace, counters, nrm, bias, after, err, st, plan.grid);
-        default: return stream_launch_th<EPI, SCALED, 32>(act, W, out, N, M, K, workspace, counters, nrm, bias, after, err, st, plan.grid);
+        case 128: return stream_launch_th<EPI, SCALED, 128>(act, W, out, N, M, K, workspace, counters, nrm, bias, after, err, st, plan.grid, groups);
+        case 64: return stream_launch_th<EPI, SCALED, 64>(act, W, out, N, M, K, workspace, counters, nrm, bias, after, err, st, plan.grid, groups);
+        default: return stream_launch_th<EPI, SCALED, 32>(act, W, out, N, M, K, workspace, counters, nrm, bias, after, err, st, plan.grid, groups);
     }
 }
 
-// mode 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out (N, M); 4: bf16 out, squared ReLU.
+// mode 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out (N, M); 4: bf16 out, squared ReLU;
+// 5: as 1 with the tanh form of gelu.
 // ssq (or null): act holds rows of a residual stream times a norm's weight and ssq ([ceil(K / 32)][16]) the sums of
 // squares of those rows by 32 columns, as mb_gemm_stream_residual leaves them: out is then the product of
 // rmsnorm(x; weight, eps).
@@ -519,8 +522,17 @@ MB_API int mb_gemm_stream(const void* act, const float* ssq, float eps, const vo
         case 1: return stream_launch<1, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
         case 2: return stream_launch<2, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
         case 4: return stream_launch<4, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
+        case 5: return stream_launch<5, false>(act, W, out, N, M, K, workspace, counters, nn, nullptr, na, err, st);
     }
     return -2;
+}
+
+// `groups` products of equal size in one launch: act (groups, N, K), W (M, K) the groups' matrices one below the other
+// (M / groups a multiple of 128), out (N, M) bf16: the columns of group g come from act[g].
+MB_API int mb_gemm_stream_groups(const void* act, const void* W, void* out, int N, int M, int K, int groups, float* workspace,
+                                 int* counters, int* err, cudaStream_t st) {
+    return stream_launch<0, false>(act, W, out, N, M, K, workspace, counters, StreamNorm{}, nullptr, StreamAfter{}, err, st,
+                                   groups);
 }
 
 // x (N, M) float32 += act (N, K) bf16 @ W (M, K)^T (+ bias (M) float32 or null), in place.  ssq_out (or null):

@@ -30,8 +30,9 @@
 
 // MODE 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out (N, M); 3: bf16 out (N, M) =
 // xIELU of the product (ap z^2 + z / 2 for z > 0, an (e^z - 1 - z) + z / 2 otherwise); 4: as 1 with the gate of routed
-// experts, g = min(gate, ap), u = clamp(up, -ap, ap), out = g sigmoid(an g) (u + shift); 5: bf16 out (N, M) = the square
-// of the product's positive part.
+// experts, g = min(gate, ap), u = clamp(up, -ap, ap), out = g sigmoid(an g) (u + shift), gate and up first times the row's
+// row_scale when that is given; 5: bf16 out (N, M) = the square of the product's positive part; 6: as 1 with the tanh form
+// of gelu on the gate.
 //
 // Grouped form (tile_expert given): W is a stack of matrices of `expert_rows` rows each, and every tile of 128 rows of
 // act belongs to one of them -- tile_expert[token tile] says which, -1: the tile holds no rows and is passed over by
@@ -42,8 +43,8 @@ __global__ void __launch_bounds__(192, 1) gemm_tc5_kernel(const __grid_constant_
                                                            const __grid_constant__ CUtensorMap wmap,
                                                            void* __restrict__ out, int N, int M, int K, float ap,
                                                            float an, float shift, int* err, const int* __restrict__ tile_expert,
-                                                           int expert_rows) {
-    constexpr bool GATED = MODE == 1 || MODE == 4;
+                                                           int expert_rows, const float* __restrict__ row_scale) {
+    constexpr bool GATED = MODE == 1 || MODE == 4 || MODE == 6;
     constexpr int FEATS = GATED ? 128 : 256;              // output features of one tile
     extern __shared__ unsigned char smem_unaligned[];
     unsigned char* smem = reinterpret_cast<unsigned char*>(
@@ -134,6 +135,7 @@ __global__ void __launch_bounds__(192, 1) gemm_tc5_kernel(const __grid_constant_
             tc_fence_after();
             const int tok = (tile % tok_tiles) * G_BM + q * 32 + lane, m0 = (tile / tok_tiles) * FEATS;
             const uint32_t taddr = tmem_base + acc * G_BN + ((uint32_t)(q * 32) << 16);
+            const float rs = MODE == 4 && row_scale && tok < N ? row_scale[tok] : 1.0f;
 #pragma unroll 1
             for (int c = 0; c < FEATS; c += 32) {
                 uint32_t r[32];
@@ -145,12 +147,16 @@ __global__ void __launch_bounds__(192, 1) gemm_tc5_kernel(const __grid_constant_
 #pragma unroll
                     for (int i = 0; i < 32; i++) {
                         // gate and up pass through bf16 as they do when the products are separate kernels
-                        float g = __bfloat162float(__float2bfloat16_rn(__uint_as_float(r[i])));
-                        float up = __bfloat162float(__float2bfloat16_rn(__uint_as_float(u[i])));
+                        float g = __bfloat162float(__float2bfloat16_rn(__uint_as_float(r[i]) * rs));
+                        float up = __bfloat162float(__float2bfloat16_rn(__uint_as_float(u[i]) * rs));
                         if (MODE == 4) {
                             g = fminf(g, ap);
                             up = fminf(fmaxf(up, -ap), ap) + shift;
                             r[i] = __float_as_uint(__fdividef(g, 1.0f + __expf(-an * g)) * up);
+                        } else if (MODE == 6) {
+                            // z / 2 (1 + tanh(y)) = z sigmoid(2 y)
+                            const float y2 = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
+                            r[i] = __float_as_uint(__fdividef(g, 1.0f + __expf(-y2)) * up);
                         } else {
                             // fast exponential and division: no slow path for huge or tiny gate values
                             r[i] = __float_as_uint(__fdividef(g, 1.0f + __expf(-g)) * up);
@@ -215,7 +221,7 @@ __global__ void __launch_bounds__(192, 1) gemm_tc5_kernel(const __grid_constant_
 template <int MODE>
 static int tc5_launch(const void* act, const void* W, void* out, int N, int M, int K, int* err, cudaStream_t st,
                       float ap = 0.0f, float an = 0.0f, const int* tile_expert = nullptr, int experts = 1,
-                      float shift = 1.0f) {
+                      float shift = 1.0f, const float* row_scale = nullptr) {
     if (N == 0 || M == 0) return 0;
     if (K % 8 || M % 8 || K < 8 || (reinterpret_cast<uintptr_t>(W) & 15) || (reinterpret_cast<uintptr_t>(act) & 15) ||
         (reinterpret_cast<uintptr_t>(out) & 15))
@@ -223,7 +229,7 @@ static int tc5_launch(const void* act, const void* W, void* out, int N, int M, i
     CUtensorMap amap, wmap;
     int rc = matrix_map(act, N, K, 128, &amap);
     if (rc) return rc;
-    constexpr int PER = (MODE == 1 || MODE == 4) ? 2 : 1;
+    constexpr int PER = (MODE == 1 || MODE == 4 || MODE == 6) ? 2 : 1;
     if (tile_expert && (experts < 1 || N % G_BM)) return -2;
     rc = matrix_map(W, (long long)PER * M * experts, K, 128, &wmap);
     if (rc) return rc;
@@ -242,7 +248,7 @@ static int tc5_launch(const void* act, const void* W, void* out, int N, int M, i
     const int feats = PER == 2 ? 128 : 256;
     const int tiles = ((N + G_BM - 1) / G_BM) * ((M + feats - 1) / feats);
     gemm_tc5_kernel<MODE><<<tiles < sms ? tiles : sms, 192, smem, st>>>(amap, wmap, out, N, M, K, ap, an, shift, err, tile_expert,
-                                                                        PER * M);
+                                                                        PER * M, row_scale);
     MB_LAUNCH_CHECK();
     return 0;
 }
@@ -256,6 +262,11 @@ MB_API int mb_gemm_tc5_bf16(const void* act, const void* W, void* out, int N, in
 MB_API int mb_gemm_tc5_swiglu_bf16(const void* act, const void* W, void* out, int N, int M, int K, int* err,
                                    cudaStream_t st) {
     return tc5_launch<1>(act, W, out, N, M, K, err, st);
+}
+// the same with the tanh form of gelu: out (N, M) = gelu_tanh(gate) * up
+MB_API int mb_gemm_tc5_geglu_bf16(const void* act, const void* W, void* out, int N, int M, int K, int* err,
+                                  cudaStream_t st) {
+    return tc5_launch<6>(act, W, out, N, M, K, err, st);
 }
 // out (N, M) = xIELU(act W^T) with the layer's two numbers as the host made them (softplus of the stored ones, the second
 // plus one half)
@@ -275,13 +286,13 @@ MB_API int mb_gemm_tc5_f32out(const void* act, const void* W, void* out, int N, 
 
 // Grouped forms: act (N, K) with N a multiple of 128, every 128 rows one expert's (tile_expert[N / 128]: its index, -1:
 // no rows); W a stack of `experts` matrices.  Gated: (experts, 2 M, K), gate rows then up rows of each expert,
-// out (N, M) bf16 = g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).
+// out (N, M) bf16 = g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit); row_scale (N
+// floats, or null): every row's gate and up are multiplied by its number first (the row's input times that number).
 MB_API int mb_gemm_tc5_grouped_gated_bf16(const void* act, const void* W, void* out, int N, int M, int K,
                                           const int* tile_expert, int experts, float limit, float alpha, float shift,
-                                          int* err,
-                                          cudaStream_t st) {
+                                          const float* row_scale, int* err, cudaStream_t st) {
     if (!tile_expert) return -2;
-    return tc5_launch<4>(act, W, out, N, M, K, err, st, limit, alpha, tile_expert, experts, shift);
+    return tc5_launch<4>(act, W, out, N, M, K, err, st, limit, alpha, tile_expert, experts, shift, row_scale);
 }
 // The same gate as a dense layer's: W (2 M, K) = [gate rows | up rows], any N; limit <= 0: no clamps.
 MB_API int mb_gemm_tc5_glu_clamped_bf16(const void* act, const void* W, void* out, int N, int M, int K, float limit,

@@ -68,6 +68,9 @@ __device__ __forceinline__ void gv_load8_stream(const float* p, float (&v)[8]) {
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
+// the modes whose W holds gate rows and up rows
+#define GV_GATED(MODE) ((MODE) == 1 || (MODE) == 6)
+
 // a product on its way to bf16: as it is, or (MODE 5) the square of its positive part, through bf16 as when the activation
 // is a kernel of its own
 template <int MODE> __device__ __forceinline__ bf16 gv_bf16(float v) {
@@ -76,8 +79,14 @@ template <int MODE> __device__ __forceinline__ bf16 gv_bf16(float v) {
     return __float2bfloat16_rn(z * z);
 }
 
+// the gated unit of two products that pass through bf16 as they do when they are separate kernels
+template <int MODE> __device__ __forceinline__ bf16 gv_gated(float gate, float up) {
+    const float g = __bfloat162float(__float2bfloat16_rn(gate)), u = __bfloat162float(__float2bfloat16_rn(up));
+    return __float2bfloat16_rn((MODE == 6 ? mb_gelu_tanh(g) : g / (1.0f + expf(-g))) * u);
+}
+
 // NT tokens (1..4).  MODE 0: bf16 out (N, M); 1: SwiGLU, W has 2 * M rows, bf16 out (N, M); 2: float out; 3: out is
-// the float32 residual stream (N, M), added to; 5: bf16 out (N, M), squared ReLU.
+// the float32 residual stream (N, M), added to; 5: bf16 out (N, M), squared ReLU; 6: as 1 with the tanh form of gelu.
 template <int NT, int MODE, int PRE>
 __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W,
                                                              void* __restrict__ out, int M, int K, GemvNorm nrm,
@@ -143,10 +152,10 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const bf16* __restr
         __syncthreads();
         act = hs;
     }
-    const int units = MODE == 1 ? M : (M + GV_ROWS - 1) / GV_ROWS;
+    const int units = GV_GATED(MODE) ? M : (M + GV_ROWS - 1) / GV_ROWS;
     for (int unit = blockIdx.x * GV_WARPS + warp; unit < units; unit += gridDim.x * GV_WARPS) {
-    int m0 = MODE == 1 ? unit : unit * GV_ROWS;                     // MODE 1: one feature (two rows); else two rows
-    int m1 = MODE == 1 ? M + m0 : min(m0 + 1, M - 1);
+    int m0 = GV_GATED(MODE) ? unit : unit * GV_ROWS;                     // MODE 1: one feature (two rows); else two rows
+    int m1 = GV_GATED(MODE) ? M + m0 : min(m0 + 1, M - 1);
     int pair = 0;                                                    // MODE 4: index of the rotated pair, -1: not rotated
     if (MODE == 4) {
         const int hh = rope.HD / 2, rh = rope.RD / 2, head = unit / hh, i = unit % hh;
@@ -254,10 +263,8 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const bf16* __restr
                     dst[m1 % rope.HD] = __float2bfloat16_rn(b);
                 }
             }
-        } else if (MODE == 1) {
-            // gate and up pass through bf16 as they do when the products are separate kernels
-            const float g = __bfloat162float(__float2bfloat16_rn(acc[0][n])), up = __bfloat162float(__float2bfloat16_rn(acc[1][n]));
-            reinterpret_cast<bf16*>(out)[(size_t)n * M + m0] = __float2bfloat16_rn((g / (1.0f + expf(-g))) * up);
+        } else if (GV_GATED(MODE)) {
+            reinterpret_cast<bf16*>(out)[(size_t)n * M + m0] = gv_gated<MODE>(acc[0][n], acc[1][n]);
         } else {
 #pragma unroll
             for (int r = 0; r < GV_ROWS; r++) {
@@ -285,10 +292,10 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_long_kernel(const bf16* __
     __shared__ float part[GV_WARPS][GV_ROWS][NT];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int unit = blockIdx.x;
-    const int m0 = MODE == 1 ? unit : unit * GV_ROWS;
+    const int m0 = GV_GATED(MODE) ? unit : unit * GV_ROWS;
     const bf16* rows[GV_ROWS];
     rows[0] = W + (size_t)m0 * K;
-    rows[1] = MODE == 1 ? W + (size_t)(M + m0) * K : W + (size_t)min(m0 + 1, M - 1) * K;
+    rows[1] = GV_GATED(MODE) ? W + (size_t)(M + m0) * K : W + (size_t)min(m0 + 1, M - 1) * K;
     float acc[GV_ROWS][NT];
 #pragma unroll
     for (int r = 0; r < GV_ROWS; r++)
@@ -340,13 +347,10 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_long_kernel(const bf16* __
     float s = 0.0f;
 #pragma unroll
     for (int w = 0; w < GV_WARPS; w++) s += part[w][r][n];            // a fixed order: the result does not depend on timing
-    if (MODE == 1) {
+    if (GV_GATED(MODE)) {
         part[0][r][n] = s;
         __syncwarp();
-        if (r == 0) {
-            const float g = __bfloat162float(__float2bfloat16_rn(part[0][0][n])), up = __bfloat162float(__float2bfloat16_rn(part[0][1][n]));
-            reinterpret_cast<bf16*>(out)[(size_t)n * M + m0] = __float2bfloat16_rn((g / (1.0f + expf(-g))) * up);
-        }
+        if (r == 0) reinterpret_cast<bf16*>(out)[(size_t)n * M + m0] = gv_gated<MODE>(part[0][0][n], part[0][1][n]);
     } else if (m0 + r < M) {
         if (MODE == 3) {
             float* xo = reinterpret_cast<float*>(out) + (size_t)n * M + m0 + r;
@@ -366,7 +370,7 @@ static int gemv_launch(const void* act, const void* W, void* out, int N, int M, 
     if (N > GV_MAX_TOKENS || K % 8 || K < 8 || (reinterpret_cast<uintptr_t>(W) & 15) ||
         (!NORM && (reinterpret_cast<uintptr_t>(act) & 15)))
         return -2;
-    const int units = MODE == 1 ? M : (M + GV_ROWS - 1) / GV_ROWS;
+    const int units = GV_GATED(MODE) ? M : (M + GV_ROWS - 1) / GV_ROWS;
     const bf16* a = (const bf16*)act;
     const bf16* w = (const bf16*)W;
     if (K >= GV_LONG_K) {
@@ -419,6 +423,10 @@ MB_API int mb_gemv_bf16(const void* act, const void* W, void* out, int N, int M,
 }
 MB_API int mb_gemv_swiglu_bf16(const void* act, const void* W, void* out, int N, int M, int K, cudaStream_t st) {
     return gemv_launch<1, false>(act, W, out, N, M, K, GemvNorm{nullptr, nullptr, 0.0f}, nullptr, st);
+}
+// the same with the tanh form of gelu
+MB_API int mb_gemv_geglu_bf16(const void* act, const void* W, void* out, int N, int M, int K, cudaStream_t st) {
+    return gemv_launch<6, false>(act, W, out, N, M, K, GemvNorm{nullptr, nullptr, 0.0f}, nullptr, st);
 }
 MB_API int mb_gemv_f32out(const void* act, const void* W, void* out, int N, int M, int K, cudaStream_t st) {
     return gemv_launch<2, false>(act, W, out, N, M, K, GemvNorm{nullptr, nullptr, 0.0f}, nullptr, st);

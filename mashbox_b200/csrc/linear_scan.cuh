@@ -3,6 +3,8 @@
 //     MODE 0 (delta rule)       S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //     MODE 1 (gated, channels)  S <- diag(g) S + k v^T;  o = S^T q          g (N, H, dim): a decay per head and key channel
 //     MODE 2 (gated, heads)     S <- g S + k v^T;  o = S^T q                g (N, H): one decay per head and token
+//     MODE 3 (wkv)              o = S^T q + b v;  S <- diag(g) S + k v^T    g as in mode 1, b (N, H): a number per head and
+//                               token (in beta's place) for what the current token alone gives
 //
 // q and k come per group (G groups, head h reads group h / (H / G)), v per head; everything float32.  See the kernel's
 // own comment for how the work is laid out.
@@ -116,9 +118,9 @@ delta_rule_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                 dr_cp4(&sv[buf][tt][c], v + ((size_t)(a + t0 + tt) * H + h) * vdim + (in ? col0 + c : 0), in ? 4 : 0);
             }
         }
-        // one number per token and head: beta of the delta rule, or the head's decay
+        // one number per token and head: beta of the delta rule, the head's decay, or the current token's share
         if (MODE != 1 && threadIdx.x < nb)
-            dr_cp4(&sb[buf][threadIdx.x], (MODE == 0 ? beta : g) + (size_t)(a + t0 + threadIdx.x) * H + h, 4);
+            dr_cp4(&sb[buf][threadIdx.x], (MODE == 2 ? g : beta) + (size_t)(a + t0 + threadIdx.x) * H + h, 4);
         asm volatile("cp.async.commit_group;\n" ::);
     };
     // every iteration commits one group (an empty one beyond the end), so the group of the stage that is worked on
@@ -165,12 +167,18 @@ delta_rule_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
                             for (int c = 0; c < CPT; c++) {
                                 const float uc = sv[buf][tt][cg * CPT + c];
                                 const uint64_t u2 = dr_pack2(uc, uc);
+                                if (MODE == 3) {                // read out before the state takes this token in
+                                    asum[c][0] = dr_fma2(st[c][r4 * 2], q01, asum[c][0]);
+                                    asum[c][1] = dr_fma2(st[c][r4 * 2 + 1], q23, asum[c][1]);
+                                }
                                 st[c][r4 * 2] = dr_fma2(st[c][r4 * 2], g01, zero2);       // the decay: a product, rounded once
                                 st[c][r4 * 2 + 1] = dr_fma2(st[c][r4 * 2 + 1], g23, zero2);
                                 st[c][r4 * 2] = dr_fma2(k01, u2, st[c][r4 * 2]);
                                 st[c][r4 * 2 + 1] = dr_fma2(k23, u2, st[c][r4 * 2 + 1]);
-                                asum[c][0] = dr_fma2(st[c][r4 * 2], q01, asum[c][0]);
-                                asum[c][1] = dr_fma2(st[c][r4 * 2 + 1], q23, asum[c][1]);
+                                if (MODE != 3) {
+                                    asum[c][0] = dr_fma2(st[c][r4 * 2], q01, asum[c][0]);
+                                    asum[c][1] = dr_fma2(st[c][r4 * 2 + 1], q23, asum[c][1]);
+                                }
                             }
                         }
 #pragma unroll
@@ -194,7 +202,8 @@ delta_rule_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
 #pragma unroll
                         for (int c = 0; c < CPT; c++)
                             if (tt0 + j < nb && colA + c < vdim)
-                                o[((size_t)(a + t0 + tt0 + j) * H + h) * vdim + colA + c] = accs[j][c];
+                                o[((size_t)(a + t0 + tt0 + j) * H + h) * vdim + colA + c] =
+                                    MODE == 3 ? fmaf(sb[buf][tt0 + j], sv[buf][tt0 + j][cg * CPT + c], accs[j][c]) : accs[j][c];
                 }
             }
         } else

@@ -8,6 +8,8 @@
 //   moe_experts    for every (token, chosen expert): g = min(Wg h, L), u = clamp(Wu h, -L, L),
 //                  y = Wd (g sigmoid(alpha g) (u + 1)), left in float32 per (token, place)
 //   moe_combine    out[n] = sum over the places, in order, of weight * y
+// The weight may meet the expert's input instead of its output (`in_wts`): gate and up, linear in the input, are multiplied
+// by it before anything else happens to them, and the sum takes the outputs as they are.
 //
 // moe_experts is the form for steps of few tokens (and of float32): blocks per (token, expert) stream that expert's
 // three matrices, which is what a decode step has to read anyway.  Dot products run over lanes with 16-byte loads where
@@ -160,7 +162,8 @@ __device__ __forceinline__ float lane_dot(const bf16* w, const float* x, int K, 
 template <typename T>
 __global__ void moe_experts_up_kernel(const T* __restrict__ h, const int* __restrict__ ids, const T* __restrict__ wg,
                                       const T* __restrict__ wu, long long gu_stride, float* __restrict__ act, int D, int F,
-                                      int E, int top, float limit, float alpha, float shift) {
+                                      int E, int top, float limit, float alpha, float shift,
+                                      const float* __restrict__ in_wts) {
     extern __shared__ float hx[];
     const int pair = blockIdx.x, j0 = blockIdx.y * MOE_ROWS;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
@@ -169,14 +172,15 @@ __global__ void moe_experts_up_kernel(const T* __restrict__ h, const int* __rest
     const T* row = h + (size_t)(pair / top) * D;
     for (int d = threadIdx.x; d < D; d += blockDim.x) hx[d] = mb_load(row + d);
     __syncthreads();
+    const float rs = in_wts ? in_wts[pair] : 1.0f;          // an expert's input times its weight: both products times it
     const T* g_rows = wg + (size_t)e * gu_stride;            // an expert's gate and up rows may lie in one tensor
     const T* u_rows = wu + (size_t)e * gu_stride;
     for (int j = j0 + warp; j < min(F, j0 + MOE_ROWS); j += nwarp) {
         float g = lane_dot(g_rows + (size_t)j * D, hx, D, lane);
         float u = lane_dot(u_rows + (size_t)j * D, hx, D, lane);
         if (lane == 0) {
-            g = fminf(g, limit);
-            u = fminf(fmaxf(u, -limit), limit);
+            g = fminf(g * rs, limit);
+            u = fminf(fmaxf(u * rs, -limit), limit);
             act[(size_t)pair * F + j] = g / (1.0f + expf(-alpha * g)) * (u + shift);
         }
     }
@@ -208,7 +212,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
     const long long n = i / D;
     const int d = (int)(i - n * D);
     float acc = 0.0f;
-    for (int kk = 0; kk < top; kk++) acc = fmaf(wts[n * top + kk], y[(n * top + kk) * D + d], acc);
+    for (int kk = 0; kk < top; kk++) acc = fmaf(wts ? wts[n * top + kk] : 1.0f, y[(n * top + kk) * D + d], acc);
     // an expert every token uses, times sigmoid of the token's gate logit (no gate: added as it is)
     if (shared) acc = fmaf(gate ? 1.0f / (1.0f + expf(-gate[n * gate_stride])) : 1.0f, mb_load(shared + i), acc);
     mb_store(out + i, acc);
@@ -230,14 +234,14 @@ MB_API int mb_moe_select(const float* z, int z_stride, const float* bias, const 
 template <typename T>
 static int moe_experts_launch(const T* h, const int* ids, const T* wg, const T* wu, long long gu_stride, const T* wd, float* y,
                               float* act, int N, int D, int F, int E, int top, float limit, float alpha, float shift,
-                              cudaStream_t st) {
+                              const float* in_wts, cudaStream_t st) {
     if (N == 0) return 0;
     const long long P = (long long)N * top;
     if (D < 1 || F < 1 || top < 1 || P > 0x7fffffff || D > 12000 || F > 12000 || (F + MOE_ROWS - 1) / MOE_ROWS > 65535 ||
         (D + MOE_ROWS - 1) / MOE_ROWS > 65535)
         return -2;
     moe_experts_up_kernel<T><<<dim3((unsigned)P, (F + MOE_ROWS - 1) / MOE_ROWS), 256, (size_t)D * sizeof(float), st>>>(
-        h, ids, wg, wu, gu_stride, act, D, F, E, top, limit, alpha, shift);
+        h, ids, wg, wu, gu_stride, act, D, F, E, top, limit, alpha, shift, in_wts);
     MB_LAUNCH_CHECK();
     moe_experts_down_kernel<T><<<dim3((unsigned)P, (D + MOE_ROWS - 1) / MOE_ROWS), 256, (size_t)F * sizeof(float), st>>>(
         act, ids, wd, y, D, F, E);
@@ -247,16 +251,16 @@ static int moe_experts_launch(const T* h, const int* ids, const T* wg, const T* 
 
 MB_API int mb_moe_experts_f32(const void* h, const int* ids, const void* wg, const void* wu, long long gu_stride,
                               const void* wd, float* y, float* act, int N, int D, int F, int E, int top, float limit,
-                              float alpha, float shift, cudaStream_t st) {
+                              float alpha, float shift, const float* in_wts, cudaStream_t st) {
     return moe_experts_launch<float>((const float*)h, ids, (const float*)wg, (const float*)wu, gu_stride, (const float*)wd, y,
-                                     act, N, D, F, E, top, limit, alpha, shift, st);
+                                     act, N, D, F, E, top, limit, alpha, shift, in_wts, st);
 }
 
 MB_API int mb_moe_experts_bf16(const void* h, const int* ids, const void* wg, const void* wu, long long gu_stride,
                                const void* wd, float* y, float* act, int N, int D, int F, int E, int top, float limit,
-                               float alpha, float shift, cudaStream_t st) {
+                               float alpha, float shift, const float* in_wts, cudaStream_t st) {
     return moe_experts_launch<bf16>((const bf16*)h, ids, (const bf16*)wg, (const bf16*)wu, gu_stride, (const bf16*)wd, y, act,
-                                    N, D, F, E, top, limit, alpha, shift, st);
+                                    N, D, F, E, top, limit, alpha, shift, in_wts, st);
 }
 
 template <typename T>
@@ -369,7 +373,7 @@ __global__ void __launch_bounds__(128)
 moe_grouped_kernel(const bf16* __restrict__ A, const bf16* __restrict__ B0, const bf16* __restrict__ B1, long long b_stride,
                    const int* __restrict__ sorted, const int* __restrict__ tiles, const int* __restrict__ n_tiles, int top,
                    int Nout, int K, bf16* __restrict__ out_act, float* __restrict__ out_y, float limit, float alpha,
-                   float shift) {
+                   float shift, const float* __restrict__ in_wts) {
     constexpr int NB = MODE == 0 ? 2 : 1;
     __shared__ __align__(16) bf16 sA[2][GG_TM][GG_LD];
     __shared__ __align__(16) bf16 sB[2][NB][GG_TN][GG_LD];
@@ -440,6 +444,7 @@ moe_grouped_kernel(const bf16* __restrict__ A, const bf16* __restrict__ B0, cons
         const int r = warp * 16 + (lane >> 2) + half * 8;
         const int pair = srow[r];
         if (pair < 0) continue;
+        const float rs = MODE == 0 && in_wts ? in_wts[pair] : 1.0f;
 #pragma unroll
         for (int j = 0; j < 8; j++)
 #pragma unroll
@@ -447,8 +452,8 @@ moe_grouped_kernel(const bf16* __restrict__ A, const bf16* __restrict__ B0, cons
                 const int n = n0 + j * 8 + (lane & 3) * 2 + x;
                 if (n >= Nout) continue;
                 if (MODE == 0) {
-                    const float g = fminf(acc[0][j][half * 2 + x], limit);
-                    const float u = fminf(fmaxf(acc[NB - 1][j][half * 2 + x], -limit), limit);
+                    const float g = fminf(acc[0][j][half * 2 + x] * rs, limit);
+                    const float u = fminf(fmaxf(acc[NB - 1][j][half * 2 + x] * rs, -limit), limit);
                     out_act[(size_t)(r0 + r) * Nout + n] = __float2bfloat16_rn(g / (1.0f + expf(-alpha * g)) * (u + shift));
                 } else {
                     out_y[(size_t)pair * Nout + n] = acc[0][j][half * 2 + x];
@@ -461,7 +466,7 @@ moe_grouped_kernel(const bf16* __restrict__ A, const bf16* __restrict__ B0, cons
 MB_API int mb_moe_grouped_bf16(const void* h, const int* ids, const void* wg, const void* wu, long long gu_stride,
                                const void* wd, float* y,
                                void* act, int* sorted, int* offsets, int* tiles, int* n_tiles, int N, int D, int F, int E,
-                               int top, float limit, float alpha, float shift, cudaStream_t st) {
+                               int top, float limit, float alpha, float shift, const float* in_wts, cudaStream_t st) {
     if (N == 0) return 0;
     const long long P = (long long)N * top;
     if (D % 8 || F % 8 || D < 8 || F < 8 || E < 1 || E > 4096 || P > (1 << 24)) return -2;
@@ -470,11 +475,11 @@ MB_API int mb_moe_grouped_bf16(const void* h, const int* ids, const void* wg, co
     MB_LAUNCH_CHECK();
     moe_grouped_kernel<0><<<dim3(max_tiles, (F + GG_TN - 1) / GG_TN), 128, 0, st>>>(
         (const bf16*)h, (const bf16*)wg, (const bf16*)wu, gu_stride, sorted, tiles, n_tiles, top, F, D, (bf16*)act, nullptr,
-        limit, alpha, shift);
+        limit, alpha, shift, in_wts);
     MB_LAUNCH_CHECK();
     moe_grouped_kernel<1><<<dim3(max_tiles, (D + GG_TN - 1) / GG_TN), 128, 0, st>>>(
         (const bf16*)act, (const bf16*)wd, nullptr, (long long)D * F, sorted, tiles, n_tiles, top, D, F, nullptr, y, limit,
-        alpha, shift);
+        alpha, shift, nullptr);
     MB_LAUNCH_CHECK();
     return 0;
 }
@@ -518,9 +523,11 @@ __global__ void moe_sort_padded_kernel(const int* __restrict__ ids, int P, int E
     }
 }
 
+// in_wts and row_scale (or null): the pair's weight goes to its place too
 __global__ void moe_gather_rows_kernel(const bf16* __restrict__ h, const int* __restrict__ place, bf16* __restrict__ rows, int D,
-                                       int top) {
+                                       int top, const float* __restrict__ in_wts, float* __restrict__ row_scale) {
     const int p = blockIdx.x;
+    if (row_scale && threadIdx.x == 0) row_scale[place[p]] = in_wts[p];
     const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)(p / top) * D);
     uint4* dst = reinterpret_cast<uint4*>(rows + (size_t)place[p] * D);
     for (int i = threadIdx.x; i < D / 8; i += blockDim.x) dst[i] = src[i];
@@ -533,7 +540,7 @@ __global__ void moe_combine_rows_kernel(const float* __restrict__ y, const int* 
     const float sg = shared ? (gate ? 1.0f / (1.0f + expf(-gate[(size_t)n * gate_stride])) : 1.0f) : 0.0f;
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
         float acc = 0.0f;
-        for (int kk = 0; kk < top; kk++) acc = fmaf(wts[(size_t)n * top + kk], y[(size_t)place[(size_t)n * top + kk] * D + d], acc);
+        for (int kk = 0; kk < top; kk++) acc = fmaf(wts ? wts[(size_t)n * top + kk] : 1.0f, y[(size_t)place[(size_t)n * top + kk] * D + d], acc);
         if (shared) acc = fmaf(sg, __bfloat162float(shared[(size_t)n * D + d]), acc);
         out[(size_t)n * D + d] = __float2bfloat16_rn(acc);
     }
@@ -541,14 +548,14 @@ __global__ void moe_combine_rows_kernel(const float* __restrict__ y, const int* 
 
 // place (N top), tile_expert (N top / 128 + E), rows ((N top / 128 + E) 128, D) bf16
 MB_API int mb_moe_sort_gather(const void* h, const int* ids, int* place, int* tile_expert, void* rows, int N, int D, int E,
-                              int top, cudaStream_t st) {
+                              int top, const float* in_wts, float* row_scale, cudaStream_t st) {
     if (N == 0) return 0;
     const long long P = (long long)N * top;
-    if (D % 8 || D < 8 || E < 1 || E > 4096 || P > (1 << 24)) return -2;
+    if (D % 8 || D < 8 || E < 1 || E > 4096 || P > (1 << 24) || (row_scale && !in_wts)) return -2;
     const int max_tiles = (int)(P / 128) + E;
     moe_sort_padded_kernel<<<1, 1024, (size_t)(2 * E + 1) * sizeof(int), st>>>(ids, (int)P, E, place, tile_expert, max_tiles);
     MB_LAUNCH_CHECK();
-    moe_gather_rows_kernel<<<(unsigned)P, 128, 0, st>>>((const bf16*)h, place, (bf16*)rows, D, top);
+    moe_gather_rows_kernel<<<(unsigned)P, 128, 0, st>>>((const bf16*)h, place, (bf16*)rows, D, top, in_wts, row_scale);
     MB_LAUNCH_CHECK();
     return 0;
 }

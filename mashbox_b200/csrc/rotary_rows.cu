@@ -8,6 +8,7 @@
 //                        the position: kpool (pages, KV, page, DK), vpool (pages, KV, page, DV).  Values mixed across
 //                        layers: v_keep receives the token's values as the product left them, (N, KV DV); with v_first
 //                        (rows kept so by another layer of the same step) what is cached is (1 - lam) v + lam v_first.
+//                        bias (as wide as q, k and v together, or null) is added to the rows first.
 //   latent_rope          the rotated strips of latent attention: of every query head (H heads of q_head values, the
 //                        strip at q_off) into the tail of that head's row of `qa` (H rows of qa_head values, the strip
 //                        at qa_off), and of the token's shared key strip (kr_off in `rows`) into the tail of the
@@ -42,7 +43,7 @@ __global__ void __launch_bounds__(NR_WARPS * 32) norm_rope_kv_write_kernel(
     const float* __restrict__ freqs, int RD, int pairing, float gain, const int* __restrict__ positions,
     const int* __restrict__ tok_row, const int* __restrict__ table, int max_blocks, T* __restrict__ kpool,
     T* __restrict__ vpool, T* __restrict__ v_keep, const T* __restrict__ v_first, float lam, int H, int KV, int DK, int DV,
-    int page, int num_pages, int* err) {
+    int page, int num_pages, int* err, const float* __restrict__ bias) {
     extern __shared__ float smem[];
     float* cs = smem;                       // cos of the RD / 2 pairs, then sin
     const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = RD / 2;
@@ -74,7 +75,12 @@ __global__ void __launch_bounds__(NR_WARPS * 32) norm_rope_kv_write_kernel(
         T* src = rows + (size_t)n * stride + (size_t)b * DK;       // the k heads follow the q heads
         const float* w = is_q ? qw : kw;
         float ss = 0.0f;
-        for (int d = lane; d < DK; d += 32) { const float x = mb_load(src + d); vals[d] = x; ss = fmaf(x, x, ss); }
+        for (int d = lane; d < DK; d += 32) {
+            float x = mb_load(src + d);
+            if (bias) x += bias[(size_t)b * DK + d];
+            vals[d] = x;
+            ss = fmaf(x, x, ss);
+        }
         if (norm_at == NR_NORM_BEFORE) {
             const float r = 1.0f / sqrtf(mb_warp_sum(ss) / (float)DK + eps);
             for (int d = lane; d < DK; d += 32) vals[d] = vals[d] * r * (w ? w[d] : 1.0f);
@@ -103,7 +109,8 @@ __global__ void __launch_bounds__(NR_WARPS * 32) norm_rope_kv_write_kernel(
                 for (int d = lane; d < DK; d += 32) mb_store(kpool + row * DK + d, vals[d]);
             const T* vs = rows + (size_t)n * stride + (size_t)(H + KV) * DK + (size_t)kvh * DV;
             for (int d = lane; d < DV; d += 32) {
-                const T v = vs[d];
+                T v = vs[d];
+                if (bias) mb_store(&v, mb_load(&v) + bias[(size_t)(H + KV) * DK + (size_t)kvh * DV + d]);
                 if (v_keep) v_keep[off + d] = v;
                 if (!have_page) continue;
                 if (v_first) mb_store(vpool + row * DV + d, (1.0f - lam) * mb_load(&v) + lam * mb_load(v_first + off + d));
@@ -134,7 +141,8 @@ __global__ void __launch_bounds__(NR_WARPS * 32) norm_rope_kv_write_quads_kernel
     T* __restrict__ rows, int stride, const float* __restrict__ qw, const float* __restrict__ kw, float eps, int norm_at,
     const float* __restrict__ freqs, int RD, float gain, const int* __restrict__ positions, const int* __restrict__ tok_row,
     const int* __restrict__ table, int max_blocks, T* __restrict__ kpool, T* __restrict__ vpool, T* __restrict__ v_keep,
-    const T* __restrict__ v_first, float lam, int H, int KV, int DK, int DV, int page, int num_pages, int* err) {
+    const T* __restrict__ v_first, float lam, int H, int KV, int DK, int DV, int page, int num_pages, int* err,
+    const float* __restrict__ bias) {
     typedef typename NrQuad<T>::type Q;
     constexpr int PER = 32 / LANES;                     // heads a warp works on at once
     extern __shared__ float2 turn[];                    // (cos, sin) of a pair
@@ -172,7 +180,12 @@ __global__ void __launch_bounds__(NR_WARPS * 32) norm_rope_kv_write_quads_kernel
         for (int i = 0; i < QUADS; i++) {
             const int d = (i * LANES + lane) * 4;
             x[i][0] = x[i][1] = x[i][2] = x[i][3] = 0.0f;
-            if (live && d < DK) nr_unpack(*reinterpret_cast<const Q*>(src + d), x[i]);
+            if (live && d < DK) {
+                nr_unpack(*reinterpret_cast<const Q*>(src + d), x[i]);
+                if (bias)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) x[i][e] += bias[(size_t)b * DK + d + e];
+            }
 #pragma unroll
             for (int e = 0; e < 4; e++) ss = fmaf(x[i][e], x[i][e], ss);
         }
@@ -227,6 +240,13 @@ __global__ void __launch_bounds__(NR_WARPS * 32) norm_rope_kv_write_quads_kernel
             const T* vs = row_n + (size_t)(H + KV) * DK + (size_t)kvh * DV;
             for (int d = lane * 4; d < DV; d += LANES * 4) {
                 Q raw = *reinterpret_cast<const Q*>(vs + d);
+                if (bias) {
+                    float a[4];
+                    nr_unpack(raw, a);
+#pragma unroll
+                    for (int e = 0; e < 4; e++) a[e] += bias[(size_t)(H + KV) * DK + (size_t)kvh * DV + d + e];
+                    nr_pack(raw, a);
+                }
                 if (v_keep) *reinterpret_cast<Q*>(v_keep + off + d) = raw;
                 if (!have_page) continue;
                 if (v_first) {
@@ -247,7 +267,8 @@ template <typename T>
 static int norm_rope_launch(T* rows, int stride, const float* qw, const float* kw, float eps, int norm_at,
                             const float* freqs, int RD, int pairing, float gain, const int* positions, const int* tok_row,
                             const int* table, int max_blocks, T* kpool, T* vpool, T* v_keep, const T* v_first, float lam,
-                            int N, int H, int KV, int DK, int DV, int page, int num_pages, int* err, cudaStream_t st) {
+                            int N, int H, int KV, int DK, int DV, int page, int num_pages, int* err, const float* bias,
+                            cudaStream_t st) {
     if (N == 0) return 0;
     if (H < 1 || KV < 1 || H + KV > 65535 * NR_WARPS || DK < 1 || DV < 1 || DK > 1024 || RD < 0 || RD > DK || (RD & 1) ||
         page < 1 || norm_at < NR_NO_NORM || norm_at > NR_NORM_AFTER)
@@ -261,7 +282,7 @@ static int norm_rope_launch(T* rows, int stride, const float* qw, const float* k
         norm_rope_kv_write_quads_kernel<T, LANES, QUADS>                                                                   \
             <<<dim3(N, N >= 592 ? 1 : passes), NR_WARPS * 32, (size_t)RD * sizeof(float), st>>>(                           \
                 rows, stride, qw, kw, eps, norm_at, freqs, RD, gain, positions, tok_row, table, max_blocks, kpool, vpool,  \
-                v_keep, v_first, lam, H, KV, DK, DV, page, num_pages, err);                                                \
+                v_keep, v_first, lam, H, KV, DK, DV, page, num_pages, err, bias);                                          \
         MB_LAUNCH_CHECK();                                                                                                 \
         return 0;                                                                                                          \
     }
@@ -271,7 +292,7 @@ static int norm_rope_launch(T* rows, int stride, const float* qw, const float* k
     norm_rope_kv_write_kernel<T><<<dim3(N, (H + KV + NR_WARPS - 1) / NR_WARPS), NR_WARPS * 32,
                                    (size_t)(RD + NR_WARPS * DK) * sizeof(float), st>>>(
         rows, stride, qw, kw, eps, norm_at, freqs, RD, pairing, gain, positions, tok_row, table, max_blocks, kpool, vpool,
-        v_keep, v_first, lam, H, KV, DK, DV, page, num_pages, err);
+        v_keep, v_first, lam, H, KV, DK, DV, page, num_pages, err, bias);
     MB_LAUNCH_CHECK();
     return 0;
 }
@@ -311,10 +332,10 @@ __global__ void latent_rope_kernel(const T* __restrict__ q, int q_stride, int q_
                                            const float* freqs, int RD, int pairing, float gain, const int* positions,      \
                                            const int* tok_row, const int* table, int max_blocks, void* kpool, void* vpool, \
                                            void* v_keep, const void* v_first, float lam, int N, int H, int KV, int DK, int DV, \
-                                           int page, int num_pages, int* err, cudaStream_t st) {                           \
+                                           int page, int num_pages, int* err, const float* bias, cudaStream_t st) {        \
         return norm_rope_launch<T>((T*)rows, stride, qw, kw, eps, norm_at, freqs, RD, pairing, gain, positions, tok_row, table, \
                                    max_blocks, (T*)kpool, (T*)vpool, (T*)v_keep, (const T*)v_first, lam, N, H, KV, DK, DV, \
-                                   page, num_pages, err, st);                                                              \
+                                   page, num_pages, err, bias, st);                                                        \
     }                                                                                                                      \
     MB_API int mb_latent_rope_##SUF(const void* q, int q_stride, int q_head, int q_off, void* qa, int qa_head, int qa_off, \
                                     const void* rows, int rows_stride, int kr_off, void* pool, int pool_row, int pool_off, \

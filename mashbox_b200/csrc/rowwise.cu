@@ -3,7 +3,8 @@
 //
 //   embed_pos        x[n] = table[token[n]] * scale + pos[position[n]]
 //   post_norm_add    x[n] += delta[n] / sqrt(mean(delta[n]^2) + eps_p) * w_p;  optionally y[n] = x[n] / sqrt(mean(x[n]^2)
-//                    + eps_n) * w_n (the norm that reads the stream next) and a copy of x[n] in the storage type
+//                    + eps_n) * w_n (the norm that reads the stream next) and a copy of x[n] in the storage type;
+//                    optionally also x[n] += again[n], a float32 row that joins the stream at this place
 //   rms_segments     two stretches of columns of a product's rows, each RMS-normed with a weight of its own: the first
 //                    goes to a buffer, the second into the cache page of the token's position (one vector per position)
 //   gated_gather     g[n, j] = gelu_tanh(z[n, j]) * table[token[n], off + j]
@@ -11,6 +12,7 @@
 //   head_product     out[n, h, j] = sum_i in[n, h, i] * W[h, i, j], W given by three strides (a projection applied
 //                    head by head from either side)
 //   scale_rows       y *= s
+//   softcap_rows     y = cap tanh(y / cap)
 #include "common.cuh"
 
 #define MB_ERR_POSITION_RANGE 5     // a position outside the learned position table
@@ -45,7 +47,7 @@ __device__ __forceinline__ void store4(bf16* p, float4 v) {
 template <typename T, bool VEC>
 __global__ void post_norm_add_kernel(float* __restrict__ x, const T* __restrict__ delta, const float* __restrict__ post_w,
                                      float post_eps, const float* __restrict__ next_w, float next_eps, T* __restrict__ normed,
-                                     T* __restrict__ copy, int D) {
+                                     T* __restrict__ copy, const float* __restrict__ again, int D) {
     extern __shared__ __align__(16) float row[];
     __shared__ float scratch[32];
     const int n = blockIdx.x;
@@ -69,7 +71,11 @@ __global__ void post_norm_add_kernel(float* __restrict__ x, const T* __restrict_
     if (VEC) {
         for (int d = threadIdx.x * 4; d < D; d += blockDim.x * 4) {
             const float4 xv = load4(x + (size_t)n * D + d), dv = load4(row + d), w = load4(post_w + d);
-            const float4 v = make_float4(xv.x + dv.x * r * w.x, xv.y + dv.y * r * w.y, xv.z + dv.z * r * w.z, xv.w + dv.w * r * w.w);
+            float4 v = make_float4(xv.x + dv.x * r * w.x, xv.y + dv.y * r * w.y, xv.z + dv.z * r * w.z, xv.w + dv.w * r * w.w);
+            if (again) {
+                const float4 a = load4(again + (size_t)n * D + d);
+                v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+            }
             store4(x + (size_t)n * D + d, v);
             store4(row + d, v);
             s2 = fmaf(v.x, v.x, s2); s2 = fmaf(v.y, v.y, s2); s2 = fmaf(v.z, v.z, s2); s2 = fmaf(v.w, v.w, s2);
@@ -77,7 +83,8 @@ __global__ void post_norm_add_kernel(float* __restrict__ x, const T* __restrict_
         }
     } else {
         for (int d = threadIdx.x; d < D; d += blockDim.x) {
-            const float v = x[(size_t)n * D + d] + row[d] * r * post_w[d];
+            float v = x[(size_t)n * D + d] + row[d] * r * post_w[d];
+            if (again) v += again[(size_t)n * D + d];
             x[(size_t)n * D + d] = v;
             row[d] = v;
             s2 = fmaf(v, v, s2);
@@ -128,10 +135,6 @@ __global__ void rms_segments_kernel(const T* __restrict__ in, int stride, int of
     for (int d = threadIdx.x; d < W; d += blockDim.x) mb_store(dst + d, mb_load(src + d) * r * w[d]);
 }
 
-__device__ __forceinline__ float gelu_tanh(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
-
 template <typename T>
 __global__ void gated_gather_kernel(const T* __restrict__ z, const int* __restrict__ tokens, const T* __restrict__ table,
                                     int table_stride, int off, T* __restrict__ out, int W, int V, int* err) {
@@ -139,7 +142,7 @@ __global__ void gated_gather_kernel(const T* __restrict__ z, const int* __restri
     int tok = tokens[n];
     if (tok < 0 || tok >= V) { if (threadIdx.x == 0) mb_set_error(err, MB_ERR_TOKEN_RANGE); tok = 0; }
     for (int j = threadIdx.x; j < W; j += blockDim.x)
-        mb_store(out + (size_t)n * W + j, gelu_tanh(mb_load(z + (size_t)n * W + j)) * mb_load(table + (size_t)tok * table_stride + off + j));
+        mb_store(out + (size_t)n * W + j, mb_gelu_tanh(mb_load(z + (size_t)n * W + j)) * mb_load(table + (size_t)tok * table_stride + off + j));
 }
 
 template <typename T>
@@ -156,11 +159,12 @@ __global__ void sigmoid_mul_kernel(T* __restrict__ o, const T* __restrict__ gate
 // (si == 1): a warp per j, lanes over i, a fixed tree.  A block per (token, head); the input row sits in shared memory.
 template <typename T, bool COLS>
 __global__ void head_product_kernel(const T* __restrict__ in, const T* __restrict__ W, T* __restrict__ out, int H, int I, int J,
-                                    long long sh, long long si, long long sj, int in_head, int out_head) {
-    // in_head, out_head: the distance between two heads of a row (a head's values may be part of a longer stretch)
+                                    long long sh, long long si, long long sj, long long in_row, int in_head, int out_head) {
+    // in_head, out_head: the distance between two heads of a row (a head's values may be part of a longer stretch); in_row:
+    // the distance between two rows of the input
     extern __shared__ float xin[];
     const int n = blockIdx.x, h = blockIdx.y;
-    for (int i = threadIdx.x; i < I; i += blockDim.x) xin[i] = mb_load(in + ((size_t)n * H + h) * in_head + i);
+    for (int i = threadIdx.x; i < I; i += blockDim.x) xin[i] = mb_load(in + (size_t)n * in_row + (size_t)h * in_head + i);
     __syncthreads();
     const T* Wh = W + (size_t)h * sh;
     T* o = out + ((size_t)n * H + h) * out_head;
@@ -186,6 +190,11 @@ __global__ void scale_rows_kernel(float* __restrict__ y, float s, long long tota
     if (i < total) y[i] *= s;
 }
 
+__global__ void softcap_rows_kernel(float* __restrict__ y, float cap, long long total) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < total) y[i] = cap * tanhf(y[i] / cap);
+}
+
 static inline int row_threads(int D) { return D >= 1024 ? 256 : D >= 256 ? 128 : 64; }
 
 template <typename T>
@@ -200,18 +209,19 @@ static int embed_pos_launch(const int* tokens, const int* positions, const T* ta
 
 template <typename T>
 static int post_norm_add_launch(float* x, const T* delta, const float* post_w, float post_eps, const float* next_w,
-                                float next_eps, T* normed, T* copy, int N, int D, cudaStream_t st) {
+                                float next_eps, T* normed, T* copy, const float* again, int N, int D, cudaStream_t st) {
     if (N == 0) return 0;
     if (D < 1 || D > 12000 || (normed && !next_w)) return -2;
     const bool vec = D % 4 == 0 && !((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(delta) |
                                      reinterpret_cast<uintptr_t>(post_w) | reinterpret_cast<uintptr_t>(next_w) |
-                                     reinterpret_cast<uintptr_t>(normed) | reinterpret_cast<uintptr_t>(copy)) & 15);
+                                     reinterpret_cast<uintptr_t>(normed) | reinterpret_cast<uintptr_t>(copy) |
+                                     reinterpret_cast<uintptr_t>(again)) & 15);
     if (vec)
         post_norm_add_kernel<T, true><<<N, D >= 2048 ? 256 : D >= 512 ? 128 : 64, (size_t)D * sizeof(float), st>>>(
-            x, delta, post_w, post_eps, next_w, next_eps, normed, copy, D);
+            x, delta, post_w, post_eps, next_w, next_eps, normed, copy, again, D);
     else
         post_norm_add_kernel<T, false><<<N, row_threads(D), (size_t)D * sizeof(float), st>>>(x, delta, post_w, post_eps, next_w,
-                                                                                             next_eps, normed, copy, D);
+                                                                                             next_eps, normed, copy, again, D);
     MB_LAUNCH_CHECK();
     return 0;
 }
@@ -254,18 +264,19 @@ static int sigmoid_mul_launch(T* o, const T* gate, int gate_stride, int N, int C
 
 template <typename T>
 static int head_product_launch(const T* in, const T* W, T* out, int N, int H, int I, int J, long long sh, long long si,
-                               long long sj, cudaStream_t st, int in_head = 0, int out_head = 0) {
+                               long long sj, cudaStream_t st, int in_head = 0, int out_head = 0, long long in_row = 0) {
     if (N == 0) return 0;
     if (in_head == 0) in_head = I;
     if (out_head == 0) out_head = J;
+    if (in_row == 0) in_row = (long long)H * in_head;
     if (H < 1 || H > 65535 || I < 1 || J < 1 || I > 12000 || (sj != 1 && si != 1) || in_head < I || out_head < J) return -2;
     const dim3 grid(N, H);
     if (sj == 1)
         head_product_kernel<T, true><<<grid, J >= 256 ? 256 : J >= 128 ? 128 : 64, (size_t)I * sizeof(float), st>>>(
-            in, W, out, H, I, J, sh, si, sj, in_head, out_head);
+            in, W, out, H, I, J, sh, si, sj, in_row, in_head, out_head);
     else
         head_product_kernel<T, false><<<grid, 256, (size_t)I * sizeof(float), st>>>(in, W, out, H, I, J, sh, si, sj,
-                                                                                    in_head, out_head);
+                                                                                    in_row, in_head, out_head);
     MB_LAUNCH_CHECK();
     return 0;
 }
@@ -276,10 +287,10 @@ static int head_product_launch(const T* in, const T* W, T* out, int N, int H, in
         return embed_pos_launch<T>(tokens, positions, (const T*)table, (const T*)pos, x, N, D, V, P, scale, err, st);      \
     }                                                                                                                     \
     MB_API int mb_post_norm_add_##SUF(float* x, const void* delta, const float* post_w, float post_eps,                  \
-                                      const float* next_w, float next_eps, void* normed, void* copy, int N, int D,        \
-                                      cudaStream_t st) {                                                                  \
-        return post_norm_add_launch<T>(x, (const T*)delta, post_w, post_eps, next_w, next_eps, (T*)normed, (T*)copy, N,   \
-                                       D, st);                                                                            \
+                                      const float* next_w, float next_eps, void* normed, void* copy, const float* again,  \
+                                      int N, int D, cudaStream_t st) {                                                    \
+        return post_norm_add_launch<T>(x, (const T*)delta, post_w, post_eps, next_w, next_eps, (T*)normed, (T*)copy,      \
+                                       again, N, D, st);                                                                            \
     }                                                                                                                     \
     MB_API int mb_rms_segments_##SUF(const void* in, int stride, int off_a, int wa, const float* w_a, void* out_a,       \
                                      int off_b, int wb, const float* w_b, void* pool, const int* positions,               \
@@ -307,10 +318,11 @@ static int head_product_launch(const T* in, const T* W, T* out, int N, int H, in
                                      long long si, long long sj, cudaStream_t st) {                                       \
         return head_product_launch<T>((const T*)in, (const T*)W, (T*)out, N, H, I, J, sh, si, sj, st);                    \
     }                                                                                                                     \
-    MB_API int mb_head_product_strided_##SUF(const void* in, int in_head, const void* W, void* out, int out_head, int N,  \
-                                             int H, int I, int J, long long sh, long long si, long long sj,               \
-                                             cudaStream_t st) {                                                           \
-        return head_product_launch<T>((const T*)in, (const T*)W, (T*)out, N, H, I, J, sh, si, sj, st, in_head, out_head); \
+    MB_API int mb_head_product_strided_##SUF(const void* in, long long in_row, int in_head, const void* W, void* out,     \
+                                             int out_head, int N, int H, int I, int J, long long sh, long long si,        \
+                                             long long sj, cudaStream_t st) {                                             \
+        return head_product_launch<T>((const T*)in, (const T*)W, (T*)out, N, H, I, J, sh, si, sj, st, in_head, out_head,  \
+                                      in_row);                                                                            \
     }
 
 ROWWISE_API(f32, float)
@@ -319,6 +331,14 @@ ROWWISE_API(bf16, bf16)
 MB_API int mb_scale_rows(float* y, float s, long long total, cudaStream_t st) {
     if (total == 0) return 0;
     scale_rows_kernel<<<(unsigned)((total + 255) / 256), 256, 0, st>>>(y, s, total);
+    MB_LAUNCH_CHECK();
+    return 0;
+}
+
+MB_API int mb_softcap_rows(float* y, float cap, long long total, cudaStream_t st) {
+    if (total == 0) return 0;
+    if (!(cap > 0.0f)) return -2;
+    softcap_rows_kernel<<<(unsigned)((total + 255) / 256), 256, 0, st>>>(y, cap, total);
     MB_LAUNCH_CHECK();
     return 0;
 }

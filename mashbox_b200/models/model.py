@@ -98,12 +98,24 @@ class Model:
         import torch
         x = ctx.ws.get("residual", ctx.N, (self.hidden,), torch.float32)
         self.embedding.forward(ctx, x)
+        start = None
+        if any(run.rejoin for run in self.schedule):        # runs before which the embedding's output joins the stream again
+            start = ctx.ws.get("embedding_kept", ctx.N, (self.hidden,), torch.float32)
+            start.copy_(x)
         pending = None
         for i, run in enumerate(self.schedule):
             # the norm that reads the stream after this block, for a block whose last product can prepare its input
             after = self.layers[self.schedule[i + 1].layer] if i + 1 < len(self.schedule) else None
             ctx.next_first_norm = after.first_norm() if hasattr(after, "first_norm") else None
+            ctx.joining = start if i + 1 < len(self.schedule) and self.schedule[i + 1].rejoin else None
+            if i == 0 and run.rejoin:
+                x.add_(start)
             pending = self.layers[run.layer].forward(ctx, x, pending, run)
+            joining = ctx.take_joining()
+            if joining is not None:         # a block that does not take it in: the sum does not mind what is pending
+                for kept in ("held", "prenormed", "stream_rows"):
+                    ctx.memo.pop(kept, None)
+                x.add_(joining)
         if ctx.n_out == 0:
             return None
         h = self.final_norm.forward(ctx, x, pending, rows=ctx.dev("want"))

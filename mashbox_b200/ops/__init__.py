@@ -290,15 +290,16 @@ def embed_positions(tokens, positions, table, pos_table, x, err, scale=1.0):
              float(scale), _p(err), _stream()), "embed_positions")
 
 
-def post_norm_add(x, delta, post_w, post_eps, next_w=None, next_eps=0.0, normed=None, copy=None):
+def post_norm_add(x, delta, post_w, post_eps, next_w=None, next_eps=0.0, normed=None, copy=None, again=None):
     """x (N, D) float32 += delta / sqrt(mean(delta^2) + post_eps) * post_w (delta in the activation dtype, post_w float32);
-    with next_w and normed: normed = x / sqrt(mean(x^2) + next_eps) * next_w; copy: x in the activation dtype"""
-    _cuda(x, delta, post_w, next_w, normed, copy)
+    with next_w and normed: normed = x / sqrt(mean(x^2) + next_eps) * next_w; copy: x in the activation dtype;
+    again (N, D) float32: added to x too"""
+    _cuda(x, delta, post_w, next_w, normed, copy, again)
     N, D = x.shape
     f = _fn("rowwise", "mb_post_norm_add_" + _suffix(delta.dtype),
-            [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p])
-    _check(f(_p(x), _p(delta), _p(post_w), float(post_eps), _p(next_w), float(next_eps), _p(normed), _p(copy), N, D,
-             _stream()), "post_norm_add")
+            [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    _check(f(_p(x), _p(delta), _p(post_w), float(post_eps), _p(next_w), float(next_eps), _p(normed), _p(copy), _p(again), N,
+             D, _stream()), "post_norm_add")
 
 
 def rms_segments(rows, off_a, w_a, out_a, off_b, w_b, pool, positions, tok_row, table, page, num_pages, eps, err):
@@ -360,9 +361,12 @@ HEAD_PRODUCT = {"tokens": 32}
 
 def head_product_strided(x, I, w, out, J, heads, transposed):
     """head_product on stretches of wider heads: x (N, heads * in_head) of whose every head the first I values are read,
-    out (N, heads * out_head) of whose every head the first J values are written; w as in head_product."""
+    out (N, heads * out_head) of whose every head the first J values are written; w as in head_product.  x may be a view
+    whose rows are further apart than they are long."""
     _cuda(x, w, out)
     N = x.shape[0]
+    if x.stride(1) != 1:
+        raise KernelError("head_product: the input's columns must be contiguous")
     in_head, out_head = x.shape[1] // heads, out.shape[1] // heads
     if tuple(w.shape) != ((heads * I, J) if transposed else (heads * J, I)) or not w.is_contiguous():
         raise KernelError("head_product: the matrix does not fit the heads")
@@ -373,8 +377,8 @@ def head_product_strided(x, I, w, out, J, heads, transposed):
         return out
     sh, si, sj = (I * J, J, 1) if transposed else (I * J, 1, I)
     f = _fn("rowwise", "mb_head_product_strided_" + _suffix(x.dtype),
-            [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_ll, c_ll, c_ll, c_void_p])
-    _check(f(_p(x), in_head, _p(w), _p(out), out_head, N, heads, I, J, sh, si, sj, _stream()), "head_product")
+            [c_void_p, c_ll, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_ll, c_ll, c_ll, c_void_p])
+    _check(f(_p(x), x.stride(0), in_head, _p(w), _p(out), out_head, N, heads, I, J, sh, si, sj, _stream()), "head_product")
     return out
 
 
@@ -404,6 +408,13 @@ def scale_rows(y, s):
     _cuda(y)
     f = _fn("rowwise", "mb_scale_rows", [c_void_p, c_float, c_ll, c_void_p])
     _check(f(_p(y), float(s), y.numel(), _stream()), "scale_rows")
+
+
+def softcap_rows(y, cap):
+    """y (float32) = cap tanh(y / cap), in place"""
+    _cuda(y)
+    f = _fn("rowwise", "mb_softcap_rows", [c_void_p, c_float, c_ll, c_void_p])
+    _check(f(_p(y), float(cap), y.numel(), _stream()), "softcap_rows")
 
 
 # ------------------------------------------------------------------------------------------------ gated delta rule
@@ -440,13 +451,13 @@ def delta_rule_lanes(lanes):
 
 def gated_rms(o, gate, w, out, H, vdim, eps, silu=False):
     """out[n, h] = o[n, h] / sqrt(mean(o[n, h]^2) + eps) * w * sigmoid(gate[n, h]) per head; o (N, H vdim) float32, gate
-    (N, H vdim) of the activation dtype whose rows may be further apart, w (vdim,) float32 or None (no weight), out the
-    activation dtype; silu: the gate is silu(gate) instead of sigmoid(gate)"""
+    (N, H vdim) of the activation dtype whose rows may be further apart, w (vdim,) float32, w (H, vdim) float32
+    (a weight per head) or None (no weight), out the activation dtype; silu: the gate is silu(gate) instead of sigmoid(gate)"""
     _cuda(o, gate, w, out)
     f = _fn("delta_rule", "mb_gated_rms_" + _suffix(out.dtype),
-            [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p])
-    _check(f(_p(o), _p(gate), gate.stride(0), 0, _p(w), _p(out), o.shape[0], H, vdim, float(eps), int(bool(silu)), _stream()),
-           "gated_rms")
+            [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p])
+    _check(f(_p(o), _p(gate), gate.stride(0), 0, _p(w), _p(out), o.shape[0], H, vdim, float(eps), int(bool(silu)),
+             vdim if w is not None and w.dim() == 2 else 0, _stream()), "gated_rms")
 
 
 # ------------------------------------------------------------------------------------------------ the stream of blocks with Dynamic Tanh
@@ -682,20 +693,21 @@ def _expert_views(wg, wu, wd):
         raise KernelError("the experts' matrices must have contiguous rows, gate and up alike")
 
 
-def moe_experts(h, ids, wg, wu, wd, y, limit, alpha, act=None, shift=1.0):
+def moe_experts(h, ids, wg, wu, wd, y, limit, alpha, act=None, shift=1.0, in_wts=None):
     """y[n, k] = Wd[e] (g sigmoid(alpha g) (u + shift)), g = min(Wg[e] h[n], limit), u = clamp(Wu[e] h[n], -limit, limit),
     e = ids[n, k].  h (N, D); wg, wu (E, F, D), whole tensors or the two halves of one (E, 2F, D) tensor; wd (E, D, F);
-    y (N, top, D) float32; act (N * top, F) float32: working memory (made here when not given)"""
-    _cuda(h, ids, wg, wu, wd, y, act)
+    y (N, top, D) float32; act (N * top, F) float32: working memory (made here when not given);
+    in_wts (N, top) float32: every expert reads h[n] times its weight"""
+    _cuda(h, ids, wg, wu, wd, y, act, in_wts)
     N, D = h.shape
     E, F, _ = wg.shape
     _expert_views(wg, wu, wd)
     if act is None:
         act = torch.empty((N * ids.shape[1], F), dtype=torch.float32, device=h.device)
     f = _fn("moe", "mb_moe_experts_" + _suffix(h.dtype),
-            [c_void_p] * 4 + [c_ll] + [c_void_p] * 3 + [c_int] * 5 + [c_float, c_float, c_float, c_void_p])
+            [c_void_p] * 4 + [c_ll] + [c_void_p] * 3 + [c_int] * 5 + [c_float, c_float, c_float, c_void_p, c_void_p])
     _check(f(_p(h), _p(ids), _p(wg), _p(wu), wg.stride(0), _p(wd), _p(y), _p(act), N, D, F, E, ids.shape[1], float(limit),
-             float(alpha), float(shift), _stream()), "moe_experts")
+             float(alpha), float(shift), _p(in_wts), _stream()), "moe_experts")
     COUNTERS["launches"] += 1
 
 
@@ -713,11 +725,11 @@ def moe_grouped_scratch(N, top, E):
     return P + (E + 1) + 3 * (P // 64 + E) + 1 + 3
 
 
-def moe_grouped(h, ids, wg, wu, wd, y, act, scratch, limit, alpha, shift=1.0):
+def moe_grouped(h, ids, wg, wu, wd, y, act, scratch, limit, alpha, shift=1.0, in_wts=None):
     """moe_experts for steps of many tokens, bf16: the (token, place) pairs are sorted by expert on the device and every
     expert's rows run through tensor-core tiles.  act (N * top, F) bf16 and scratch (moe_grouped_scratch values, int32)
     are working memory."""
-    _cuda(h, ids, wg, wu, wd, y, act, scratch)
+    _cuda(h, ids, wg, wu, wd, y, act, scratch, in_wts)
     N, D = h.shape
     E, F, _ = wg.shape
     top = ids.shape[1]
@@ -729,9 +741,10 @@ def moe_grouped(h, ids, wg, wu, wd, y, act, scratch, limit, alpha, shift=1.0):
     tiles = scratch[P + E + 1:P + E + 1 + 3 * max_tiles]
     n_tiles = scratch[P + E + 1 + 3 * max_tiles:]
     _expert_views(wg, wu, wd)
-    f = _fn("moe", "mb_moe_grouped_bf16", [c_void_p] * 4 + [c_ll] + [c_void_p] * 7 + [c_int] * 5 + [c_float, c_float, c_float, c_void_p])
+    f = _fn("moe", "mb_moe_grouped_bf16", [c_void_p] * 4 + [c_ll] + [c_void_p] * 7 + [c_int] * 5 + [c_float, c_float, c_float, c_void_p, c_void_p])
     _check(f(_p(h), _p(ids), _p(wg), _p(wu), wg.stride(0), _p(wd), _p(y), _p(act), _p(sorted_), _p(offsets), _p(tiles),
-             _p(n_tiles), N, D, F, E, top, float(limit), float(alpha), float(shift), _stream()), "moe_grouped")
+             _p(n_tiles), N, D, F, E, top, float(limit), float(alpha), float(shift), _p(in_wts),
+             _stream()), "moe_grouped")
     COUNTERS["launches"] += 2
 
 
@@ -745,37 +758,40 @@ def moe_tc5_tiles(N, top, E):
     return N * top // 128 + E
 
 
-def moe_tc5(h, ids, wts, wgu, wd, out, rows, act, y, scratch, limit, alpha, shift=1.0, shared=None, gate=None):
+def moe_tc5(h, ids, wts, wgu, wd, out, rows, act, y, scratch, limit, alpha, shift=1.0, shared=None, gate=None,
+            row_scale=None):
     """The routed experts of a step of many tokens, bf16: ids (N, top) and wts from moe_select; wgu (E, 2F, D), every
     expert's gate rows then its up rows; wd (E, D, F); out (N, D).  Working memory, with T = moe_tc5_tiles(N, top, E):
     rows (128 T, D) bf16, act (128 T, F) bf16, y (128 T, D) float32, scratch (N top + T) int32.  shared (N, D) and gate
-    (float32, one logit per token, rows gate.stride(0) apart): see moe_combine."""
-    _cuda(h, ids, wts, wgu, wd, out, rows, act, y, scratch, shared, gate)
+    (float32, one logit per token, rows gate.stride(0) apart): see moe_combine.  row_scale (128 T float32, working memory): the
+    weights meet the experts' inputs instead of their outputs."""
+    _cuda(h, ids, wts, wgu, wd, out, rows, act, y, scratch, shared, gate, row_scale)
     N, D = h.shape
     E, F = wgu.shape[0], wgu.shape[1] // 2
     top = ids.shape[1]
     T = moe_tc5_tiles(N, top, E)
-    if rows.shape[0] < 128 * T or act.shape[0] < 128 * T or y.shape[0] < 128 * T or scratch.numel() < N * top + T:
+    if rows.shape[0] < 128 * T or act.shape[0] < 128 * T or y.shape[0] < 128 * T or scratch.numel() < N * top + T \
+            or (row_scale is not None and row_scale.numel() < 128 * T):
         raise KernelError("moe_tc5: the working memory is too small")
     place, tile_expert = scratch[:N * top], scratch[N * top:N * top + T]
-    f = _fn("moe", "mb_moe_sort_gather", [c_void_p] * 5 + [c_int] * 4 + [c_void_p])
-    _check(f(_p(h), _p(ids), _p(place), _p(tile_expert), _p(rows), N, D, E, top, _stream()), "moe_sort_gather")
+    f = _fn("moe", "mb_moe_sort_gather", [c_void_p] * 5 + [c_int] * 4 + [c_void_p] * 3)
+    _check(f(_p(h), _p(ids), _p(place), _p(tile_expert), _p(rows), N, D, E, top, _p(wts), _p(row_scale), _stream()),
+           "moe_sort_gather")
     err = error_word(h.device)
     f = _fn("gemm_tc5", "mb_gemm_tc5_grouped_gated_bf16",
-            [c_void_p] * 3 + [c_int] * 3 + [c_void_p, c_int, c_float, c_float, c_float, c_void_p, c_void_p])
-    _check(f(_p(rows), _p(wgu), _p(act), 128 * T, F, D, _p(tile_expert), E, float(limit), float(alpha), float(shift), _p(err),
-             _stream()),
-           "gemm_tc5_grouped_gated")
+            [c_void_p] * 3 + [c_int] * 3 + [c_void_p, c_int, c_float, c_float, c_float, c_void_p, c_void_p, c_void_p])
+    _check(f(_p(rows), _p(wgu), _p(act), 128 * T, F, D, _p(tile_expert), E, float(limit), float(alpha), float(shift),
+             _p(row_scale), _p(err), _stream()), "gemm_tc5_grouped_gated")
     f = _fn("gemm_tc5", "mb_gemm_tc5_grouped_f32out", [c_void_p] * 3 + [c_int] * 3 + [c_void_p, c_int, c_void_p, c_void_p])
     _check(f(_p(act), _p(wd), _p(y), 128 * T, D, F, _p(tile_expert), E, _p(err), _stream()), "gemm_tc5_grouped")
     f = _fn("moe", "mb_moe_combine_rows", [c_void_p] * 4 + [c_int] * 3 + [c_void_p, c_void_p, c_int, c_void_p])
-    _check(f(_p(y), _p(place), _p(wts), _p(out), N, D, top, _p(shared), _p(gate), gate.stride(0) if gate is not None else 0,
+    _check(f(_p(y), _p(place), _p(wts if row_scale is None else None), _p(out), N, D, top, _p(shared), _p(gate), gate.stride(0) if gate is not None else 0,
              _stream()), "moe_combine_rows")
     COUNTERS["launches"] += 1
 
 
 def moe_combine(y, wts, out, shared=None, gate=None):
-    """out[n] = sum_k wts[n, k] y[n, k] (places in order); y (N, top, D) float32, out (N, D) the activation dtype.
+    """out[n] = sum_k wts[n, k] y[n, k] (places in order; wts None: every weight 1); y (N, top, D) float32, out (N, D) the activation dtype.
     shared (N, D) of the activation dtype: the output of an expert every token uses, added times sigmoid(gate[n]) (gate:
     float32, one logit per token, rows gate.stride(0) apart; None: added as it is)"""
     _cuda(y, wts, out, shared, gate)
@@ -794,8 +810,8 @@ def linear(a, w, out=None, out_dtype=None):
     if a.dtype == torch.float32:
         if out is None:
             out = torch.empty((N, M), dtype=torch.float32, device=a.device)
-        f = _fn("gemm_f32", "mb_gemm_f32", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
-        _check(f(_p(a), _p(w), _p(out), N, M, K, _stream()), "gemm_f32")
+        f = _fn("gemm_f32", "mb_gemm_f32", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+        _check(f(_p(a), _p(w), _p(out), N, M, K, out.stride(0) if N > 1 else M, _stream()), "gemm_f32")
         return out
     if tc5_supports(N, M, K) and a.is_contiguous() and w.is_contiguous() and a.dtype == torch.bfloat16:
         want = a.dtype if out_dtype is None else out_dtype
@@ -826,6 +842,23 @@ def linear(a, w, out=None, out_dtype=None):
     return torch.mm(a, w.t())
 
 
+def linear_groups(a, w, out):
+    """Products of equal size side by side: a (G, N, K), w (G M, K) = the groups' matrices one below the other, out (N, G M):
+    columns g M .. (g + 1) M are a[g] w[g]^T.  One launch for decode steps whose sizes the weight-streaming product takes."""
+    _cuda(a, w, out)
+    G, N, K = a.shape
+    M = w.shape[0] // G
+    if a.dtype == torch.bfloat16 and stream_supports(N, K) and M % 128 == 0:
+        ws, cnt = _stream_buffers(a.device, G * M)
+        f = _fn("gemm_stream", "mb_gemm_stream_groups", [c_void_p] * 3 + [c_int] * 4 + [c_void_p] * 4)
+        _check(f(_p(a), _p(w), _p(out), N, G * M, K, G, _p(ws), _p(cnt), _p(error_word(a.device)), _stream()),
+               "gemm_stream_groups")
+        return out
+    for g in range(G):
+        linear(a[g], w[g * M:(g + 1) * M], out=out[:, g * M:(g + 1) * M])
+    return out
+
+
 # The package's own tcgen05 product for prompt portions (128 tokens or more).  "swiglu": the fused gate/up product
 # (measured 317 us against 310 + 33 us for the library product and the separate gate kernel at 2,048 tokens of the
 # Llama-3.1-8B shape); "plain": every product (87 to 97 % of the library's speed, so off by default).
@@ -841,7 +874,8 @@ def linear_tc5(a, w, out, mode="plain"):
     "swiglu" (silu(gate) * up), float32 for "float".  TMA + tcgen05.mma with the accumulator in tensor memory."""
     _cuda(a, w, out)
     N, K = a.shape
-    name = {"plain": "mb_gemm_tc5_bf16", "swiglu": "mb_gemm_tc5_swiglu_bf16", "float": "mb_gemm_tc5_f32out"}[mode]
+    name = {"plain": "mb_gemm_tc5_bf16", "swiglu": "mb_gemm_tc5_swiglu_bf16", "geglu": "mb_gemm_tc5_geglu_bf16",
+            "float": "mb_gemm_tc5_f32out"}[mode]
     f = _fn("gemm_tc5", name, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(f(_p(a), _p(w), _p(out), N, out.shape[1], K, _p(error_word(a.device)), _stream()), "gemm_tc5")
     return out
@@ -923,7 +957,7 @@ def linear_gemv(a, w, out, mode="plain"):
     _cuda(a, w, out)
     N, K = a.shape
     name = {"plain": "mb_gemv_bf16", "swiglu": "mb_gemv_swiglu_bf16", "float": "mb_gemv_f32out",
-            "relu2": "mb_gemv_relu2_bf16"}[mode]
+            "relu2": "mb_gemv_relu2_bf16", "geglu": "mb_gemv_geglu_bf16"}[mode]
     f = _fn("gemv", name, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(f(_p(a), _p(w), _p(out), N, out.shape[1], K, _stream()), "gemv")
     return out
@@ -991,7 +1025,7 @@ def linear_stream(a, w, out, mode="plain", sums=None, eps=0.0):
     ws, cnt = _stream_buffers(a.device, M)
     f = _fn("gemm_stream", "mb_gemm_stream", [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                               c_void_p, c_void_p, c_void_p, c_void_p])
-    _check(f(_p(a), _p(sums), float(eps), _p(w), _p(out), N, M, K, {"plain": 0, "swiglu": 1, "float": 2, "relu2": 4}[mode], _p(ws),
+    _check(f(_p(a), _p(sums), float(eps), _p(w), _p(out), N, M, K, {"plain": 0, "swiglu": 1, "float": 2, "relu2": 4, "geglu": 5}[mode], _p(ws),
              _p(cnt), _p(error_word(a.device)), _stream()), "gemm_stream")
     return out
 
@@ -1052,6 +1086,13 @@ def linear_small_residual(a, w, x, bias=None, sums=None, next_w=None, scaled=Non
         return False
     linear_stream_residual(a, w, x, bias, sums, next_w, scaled)
     return sums is not None and scaled is not None
+
+
+def geglu(gu, out):
+    """gu (N, 2F) = [gate | up] -> out (N, F) = gelu_tanh(gate) * up"""
+    _cuda(gu, out)
+    f = _fn("elementwise", "mb_geglu_" + _suffix(out.dtype), [c_void_p, c_void_p, c_int, c_int, c_void_p])
+    _check(f(_p(gu), _p(out), out.shape[0], out.shape[1], _stream()), "geglu")
 
 
 def fused_swiglu_supports(N, F, K):
@@ -1115,18 +1156,19 @@ def linear_glu_clamped(a, wgu, out, limit, alpha=1.702, shift=1.0):
     return out
 
 
-def linear_swiglu(a, wgu, out):
-    """a (N, K) bf16, wgu (2F, K) = [gate rows | up rows] -> out (N, F) = silu(a Wg^T) * (a Wu^T), one kernel: the
+def linear_swiglu(a, wgu, out, mode="swiglu"):
+    """a (N, K) bf16, wgu (2F, K) = [gate rows | up rows] -> out (N, F) = silu(a Wg^T) * (a Wu^T) (mode "geglu": the tanh
+    form of gelu in silu's place), one kernel: the
     tcgen05 product for prompt portions, the matrix-vector or the weight-streaming kernel for decode batches (where enabled).
     Only for shapes fused_swiglu_supports() takes."""
     _cuda(a, wgu, out)
     N, K = a.shape
     if tc5_supports(N, out.shape[1], K, "swiglu"):
-        return linear_tc5(a, wgu, out, "swiglu")
+        return linear_tc5(a, wgu, out, mode)
     if gemv_supports(N, K, "swiglu"):
-        return linear_gemv(a, wgu, out, "swiglu")
+        return linear_gemv(a, wgu, out, mode)
     if stream_supports(N, K):
-        return linear_stream(a, wgu, out, "swiglu")
+        return linear_stream(a, wgu, out, mode)
     raise KernelError("linear_swiglu: no fused kernel takes these sizes")
 
 
@@ -1276,9 +1318,10 @@ def attention_tma_active_clusters(HD, cluster):
 
 def attention_tma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_start, q_len, pos0, part_base, seq_row,
                   table, part_o, part_ml, max_splits, H, KV, HD, page, num_pages, window, scale, err, merge=False,
-                  rope=None, cluster=0, keep=0):
+                  rope=None, cluster=0, keep=0, sinks=None):
     """The same contract as attention_mma, with K/V tiles loaded by TMA (head sizes 64 and 128, pages of 8 to 64).
-    keep: behind the window the first `keep` positions stay visible.
+    keep: behind the window the first `keep` positions stay visible.  sinks (H,) float32: a score per query head that joins
+    the softmax's denominator without a value.
     merge: the last block of every split group merges the group's partial results and writes `out`, so no
     attention_merge is needed afterwards (only when attention_tma_merges(n_items, KV)).
     cluster = n > 1 (decode form): every sequence of the launch is cut into n splits and the blocks of a sequence and kv
@@ -1287,7 +1330,7 @@ def attention_tma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_star
     rope = (bias or None, freqs or None, RD, pairing): the step's sequences bring ONE token each and q is the whole
     (N, (H + 2 KV) HD) output of the q/k/v product; the kernel does what rope_kv_write would have done before it (bias,
     rotation of q and k, k and v into the token's page) -- the same bits, one launch fewer.  q itself is not changed."""
-    _cuda(q, out, kpool, vpool, items, q_start, q_len, pos0, part_base, table, part_o, part_ml)
+    _cuda(q, out, kpool, vpool, items, q_start, q_len, pos0, part_base, table, part_o, part_ml, sinks)
     if cluster and cluster > 1:
         if not decode:
             raise KernelError("attention_tma: clusters are for the decode form")
@@ -1295,10 +1338,10 @@ def attention_tma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_star
         _cuda(bias, freqs)
         f = _fn("attention_tma", "mb_attn_tma_cluster_bf16",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                 c_void_p, c_int] + [c_int] * 8 + [c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
+                 c_void_p, c_int] + [c_int] * 8 + [c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
         code = f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, _p(q_start), _p(q_len), _p(pos0),
                  _p(seq_row), _p(table), table.shape[1], int(cluster), H, KV, HD, page, num_pages, window or 0, int(keep),
-                 float(scale), _p(err), 1 if rope is not None else 0, _p(bias), _p(freqs), int(RD), int(pairing), _stream())
+                 _p(sinks), float(scale), _p(err), 1 if rope is not None else 0, _p(bias), _p(freqs), int(RD), int(pairing), _stream())
         if code == -6:
             raise KernelError("attention_tma: the driver refused the tensor map of the cache pool")
         _check(code, "attention_tma")
@@ -1319,19 +1362,20 @@ def attention_tma(q, q_stride, out, kpool, vpool, items, n_items, decode, q_star
         _cuda(bias, freqs)
         f = _fn("attention_tma", "mb_attn_tma_rope_bf16",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                 c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_void_p, c_void_p, c_void_p,
-                                                                                c_void_p, c_int, c_int, c_void_p])
+                 c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_float, c_void_p, c_void_p,
+                                                                                c_void_p, c_void_p, c_int, c_int, c_void_p])
         code = f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, _p(q_start), _p(q_len), _p(pos0),
                  _p(part_base), _p(seq_row), _p(table), table.shape[1], _p(part_o), _p(part_ml), max_splits, H, KV, HD,
-                 page, num_pages, window or 0, int(keep), float(scale), _p(counters), _p(err), _p(bias), _p(freqs), int(RD),
+                 page, num_pages, window or 0, int(keep), _p(sinks), float(scale), _p(counters), _p(err), _p(bias), _p(freqs), int(RD),
                  int(pairing), _stream())
     else:
         f = _fn("attention_tma", "mb_attn_tma_bf16",
                 [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                 c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8 + [c_float, c_void_p, c_void_p, c_void_p])
+                 c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p] + [c_int] * 8 + [c_void_p, c_float, c_void_p, c_void_p, c_void_p])
         code = f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, 1 if decode else 0, _p(q_start),
                  _p(q_len), _p(pos0), _p(part_base), _p(seq_row), _p(table), table.shape[1], _p(part_o), _p(part_ml),
-                 max_splits, H, KV, HD, page, num_pages, window or 0, int(keep), float(scale), _p(counters), _p(err), _stream())
+                 max_splits, H, KV, HD, page, num_pages, window or 0, int(keep), _p(sinks), float(scale), _p(counters), _p(err),
+                 _stream())
     if code == -6:
         raise KernelError("attention_tma: the driver refused the tensor map of the cache pool")
     _check(code, "attention_tma")
@@ -1349,16 +1393,17 @@ def attention_tc5_rows():
 
 
 def attention_tc5(q, q_stride, out, kpool, vpool, items, n_items, q_start, q_len, pos0, seq_row, table, H, KV, HD, page,
-                  num_pages, window, scale, err, keep=0):
+                  num_pages, window, scale, err, keep=0, sinks=None):
     """Prompt-form attention on tcgen05: items are (sequence, tile of attention_tc5_rows() packed rows, 0, 1); head
-    sizes 64 and 128.  keep: behind the window the first `keep` positions stay visible."""
-    _cuda(q, out, kpool, vpool, items, q_start, q_len, pos0, seq_row, table)
+    sizes 64 and 128.  keep: behind the window the first `keep` positions stay visible.  sinks (H,) float32: a score per
+    query head that joins the softmax's denominator without a value."""
+    _cuda(q, out, kpool, vpool, items, q_start, q_len, pos0, seq_row, table, sinks)
     f = _fn("attention_tc5", "mb_attn_tc5_bf16",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-             c_void_p, c_int] + [c_int] * 6 + [c_float, c_int, c_void_p, c_void_p])
+             c_void_p, c_int] + [c_int] * 6 + [c_float, c_int, c_void_p, c_void_p, c_void_p])
     _check(f(_p(q), q_stride, _p(out), _p(kpool), _p(vpool), _p(items), n_items, _p(q_start), _p(q_len), _p(pos0),
              _p(seq_row), _p(table), table.shape[1], H, KV, HD, page, num_pages, window or 0, float(scale), int(keep),
-             _p(err), _stream()), "attention_tc5")
+             _p(sinks), _p(err), _stream()), "attention_tc5")
 
 
 def attention_tc5_diff_supports(dim, vdim, page):
@@ -1543,35 +1588,66 @@ def ssd_out(o, xbc, conv_bias, D, z, w, out, H, P, parts, eps):
              parts, float(eps), _stream()), "ssd_out")
 
 
-def gated_scan(q, k, v, g, o, state, seq, H, G, dim, vdim, per_head):
+def gated_scan(q, k, v, g, o, state, seq, H, G, dim, vdim, per_head, bonus=None):
     """S <- decay S + k v^T, o = S^T q per head and token, tokens of a sequence in order.  q, k (N, G dim), v (N, H vdim),
     o (N, H vdim) float32; g (N, H dim) a decay per key channel, or (N, H) with per_head; state (slots, H dim vdim)
-    float32 (a view: slots state.stride(0) apart); seq = (q_start, q_len, state_slot) int32 device arrays"""
-    _cuda(q, k, v, g, o, state, *seq)
-    f = _fn("gated_scan", "mb_gated_scan", [c_void_p] * 6 + [c_ll] + [c_void_p] * 3 + [c_int] * 7 + [c_void_p])
+    float32 (a view: slots state.stride(0) apart); seq = (q_start, q_len, state_slot) int32 device arrays.
+    bonus (N, H) float32 (decays per channel): o = S^T q + bonus v BEFORE the token joins the state"""
+    _cuda(q, k, v, g, o, state, bonus, *seq)
+    f = _fn("gated_scan", "mb_gated_scan", [c_void_p] * 7 + [c_ll] + [c_void_p] * 3 + [c_int] * 7 + [c_void_p])
     S = seq[0].shape[0]
     # which layout of the state over threads: by the step's tokens per sequence (from the lengths of the arrays alone)
-    _check(f(_p(q), _p(k), _p(v), _p(g), _p(o), _p(state), state.stride(0), *[_p(t) for t in seq], S, H, G,
+    _check(f(_p(q), _p(k), _p(v), _p(g), _p(bonus), _p(o), _p(state), state.stride(0), *[_p(t) for t in seq], S, H, G,
              dim, vdim, 1 if per_head else 0, 1 if q.shape[0] > 4 * S else 0, _stream()), "gated_scan")
+
+
+def token_mix(h, mu, state, seq, out):
+    """out[s, n] = h[n] + (h' - h[n]) mu[s], h' the row of the token before n in its sequence: h[n - 1], or for a sequence's
+    first token of the step what `state` keeps of it (zeros at its start), which the sequence's last row then replaces.
+    h (N, D), out (streams, N, D) of the activation dtype, mu (streams, D) float32, state (slots, D) float32 (a view, slots
+    state.stride(0) apart); seq = (tok_seq, q_start, q_len, state_slot) int32 device arrays"""
+    _cuda(h, mu, state, out, *seq)
+    N, D = h.shape
+    f = _fn("wkv", "mb_token_mix_" + _suffix(h.dtype), [c_void_p] * 7 + [c_ll, c_void_p] + [c_int] * 3 + [c_void_p])
+    _check(f(_p(h), _p(mu), *[_p(t) for t in seq], _p(state), state.stride(0), _p(out), N, D, mu.shape[0], _stream()),
+           "token_mix")
+
+
+def tanh_rows(x, out):
+    """out = tanh(x), x float32, out of the activation dtype"""
+    _cuda(x, out)
+    f = _fn("wkv", "mb_tanh_rows_" + _suffix(out.dtype), [c_void_p, c_void_p, c_ll, c_void_p])
+    _check(f(_p(x), _p(out), x.numel(), _stream()), "tanh_rows")
+
+
+def wkv_gates(rows, w0, u, r, k, v, g, b, H, dim, z=None, low=None, w2=None):
+    """rows (N, >= 3 H dim) = [r | k | v | ..] in the activation dtype -> float32 r, k, v (N, H dim), the decay
+    g = exp(-exp(z + w0)) (N, H dim) and b = sum over a head of r u k (N, H).  z (N, H dim) float32, or low (N, R) float32
+    and w2 (H dim, R): z = W2 tanh(low), made in the kernel."""
+    _cuda(rows, w0, u, r, k, v, g, b, z, low, w2)
+    f = _fn("wkv", "mb_wkv_gates_" + _suffix(rows.dtype),
+            [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int] + [c_void_p] * 7 + [c_int] * 3 + [c_void_p])
+    _check(f(_p(rows), rows.stride(0), _p(z), _p(low), _p(w2), low.shape[1] if low is not None else 0, _p(w0), _p(u), _p(r),
+             _p(k), _p(v), _p(g), _p(b), rows.shape[0], H, dim, _stream()), "wkv_gates")
 
 
 # ------------------------------------------------------------------------------------------------ normed, rotated heads
 def norm_rope_kv_write(rows, qw, kw, eps, freqs, RD, pairing, gain, positions, tok_row, table, kpool, vpool, H, KV, DK,
-                       DV, page, num_pages, err, norm="before", v_keep=None, v_first=None, lam=0.0):
+                       DV, page, num_pages, err, norm="before", v_keep=None, v_first=None, lam=0.0, bias=None):
     """rows (N, >= (H + KV) DK + KV DV) = [q | k | v | ..]: the first RD values of every q and k head rotated by the token's
     position (freqs (RD/2,) float32 or None; pairing 0 adjacent, 1 halves; cos and sin times gain), the head divided by its
     root mean square and multiplied by qw / kw (DK values; None: no weights) before or after that (norm: "before" |
     "after" | None); q back in place, k and v into the pages: kpool (pages, KV, page, DK), vpool (pages, KV, page, DV); both
     None: q only.  v_keep (N, KV DV): receives the values as they are; v_first (N, KV DV): what is cached is
-    (1 - lam) v + lam v_first."""
-    _cuda(rows, qw, kw, freqs, positions, tok_row, table, kpool, vpool, v_keep, v_first)
+    (1 - lam) v + lam v_first.  bias ((H + KV) DK + KV DV,) float32: added to q, k and v first."""
+    _cuda(rows, qw, kw, freqs, positions, tok_row, table, kpool, vpool, v_keep, v_first, bias)
     f = _fn("rotary_rows", "mb_norm_rope_kv_write_" + _suffix(rows.dtype),
             [c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
-             c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float] + [c_int] * 7 + [c_void_p, c_void_p])
+             c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float] + [c_int] * 7 + [c_void_p, c_void_p, c_void_p])
     _check(f(_p(rows), rows.stride(0), _p(qw), _p(kw), float(eps), {None: 0, "before": 1, "after": 2}[norm], _p(freqs),
              int(RD), int(pairing), float(gain), _p(positions), _p(tok_row), _p(table), table.shape[1], _p(kpool), _p(vpool),
-             _p(v_keep), _p(v_first), float(lam), rows.shape[0], H, KV, DK, DV, page, num_pages, _p(err), _stream()),
-           "norm_rope_kv_write")
+             _p(v_keep), _p(v_first), float(lam), rows.shape[0], H, KV, DK, DV, page, num_pages, _p(err), _p(bias),
+             _stream()), "norm_rope_kv_write")
 
 
 def latent_rope(q, q_head, q_off, qa, qa_head, qa_off, rows, kr_off, pool, pool_off, freqs, RD, W, pairing, gain,

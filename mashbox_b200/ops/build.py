@@ -38,6 +38,7 @@ LIBRARIES = {            # library name -> (source file, extra compiler flags)
     "rowwise": ("rowwise.cu", []),                                     # learned positions, norms of sublayer outputs, latents
     "delta_rule": ("delta_rule.cu", []),                               # the gated delta rule and what feeds it
     "gated_scan": ("gated_scan.cu", []),                               # gated linear attention, state-space duality
+    "wkv": ("wkv.cu", []),                                             # what feeds the wkv recurrence
     "layernorm": ("layernorm.cu", []),                                 # layer norm of sublayer outputs and of the stream
     "rotary_rows": ("rotary_rows.cu", []),                             # head norms, rotation of strips, cache writes
     "moe": ("moe.cu", []),                                             # routed experts

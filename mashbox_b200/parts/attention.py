@@ -57,10 +57,10 @@ class PagedAttention:
         """vdim: the width of a value when it is not the key's (the result is heads * vdim wide); softcap: scores become
         softcap tanh(s / softcap); sinks: attend() is handed one number per query head that joins the softmax's
         denominator without a value; gated: attend() is handed a gate per token and query head (the head's result
-        times its sigmoid).  Any of the four, or pools whose rows are wider than what is read of them, make the
-        attention *general*: it runs on the kernels that take all of that.  keep_first: behind the window the first
-        `keep_first` positions stay visible, which the TMA and tcgen05 kernels take and the general ones; where a step
-        would run another kernel the attention is general too (`is_general`)."""
+        times its sigmoid).  Other value widths, a cap, gates, or pools whose rows are wider than what is read of them,
+        make the attention *general*: it runs on the kernels that take all of that.  keep_first: behind the window the
+        first `keep_first` positions stay visible.  That and sinks the TMA and tcgen05 kernels take, and the general ones;
+        where a step would run another kernel the attention is general too (`is_general`)."""
         self.H, self.KV, self.HD = int(heads), int(kv_heads), int(head_dim)
         if self.H % self.KV:
             raise ConfigError(f"{heads} heads do not divide into {kv_heads} kv heads")
@@ -69,13 +69,14 @@ class PagedAttention:
         self.VD = int(vdim) if vdim else self.HD
         self.softcap = float(softcap) if softcap else None
         self.keep = int(keep_first) if self.window else 0       # without a window every position is visible anyway
-        self.general = self.VD != self.HD or self.softcap is not None or bool(sinks) or bool(gated)
+        self.sunk = bool(sinks)
+        self.general = self.VD != self.HD or self.softcap is not None or bool(gated)
 
     # ------------------------------------------------------------------------------------------ planning
     def is_general(self, ctx):
         """whether this step runs the general kernels"""
         import torch
-        if self.general or not self.keep:
+        if self.general or not (self.keep or self.sunk):
             return self.general
         page = ctx.cache.page_size
         return not (ctx.dtype == torch.bfloat16 and ctx.options.get("attention_kernel", "tma") == "tma"
@@ -102,7 +103,7 @@ class PagedAttention:
 
     def plan_key(self):
         # everything the work list depends on: the head size decides the kernel and its rows per tile
-        return ("attention", self.H // self.KV, self.KV, self.HD, self.window, self.keep, self.general)
+        return ("attention", self.H // self.KV, self.KV, self.HD, self.window, self.keep, self.general, self.sunk)
 
     def prepare(self, ctx):
         """Work list of the flash kernel for this step: (sequence, row tile, split, splits) per block, decode-form
@@ -233,19 +234,22 @@ class PagedAttention:
             extra = dict(merge=True) if fused else {}
             if self.keep:
                 extra["keep"] = self.keep
+            if self.sunk:
+                extra["sinks"] = sinks
             if rope is not None:
                 extra["rope"] = rope
             if plan["tc5"] and plan["n_pre"]:
                 ops.attention_tc5(qkv, width, out, kpool, vpool, ctx.dev(nm + "pre"), plan["n_pre"], ctx.dev("q_start"),
                                   ctx.dev("q_len"), ctx.dev("pos0"), ctx.dev("seq_row"), table, H, KV, HD, page, pages,
-                                  self.window, self.scale, ctx.err, keep=self.keep)
+                                  self.window, self.scale, ctx.err, keep=self.keep, sinks=sinks if self.sunk else None)
             for form, n_items, decode in ((nm + "pre", 0 if plan["tc5"] else plan["n_pre"], False),
                                           (nm + "mid", plan["n_mid"], False), (nm + "dec", plan["n_dec"], True)):
                 if n_items and decode and plan["cluster"]:
                     ops.attention_tma(qkv, width, out, kpool, vpool, ctx.dev(form), n_items, True, ctx.dev("q_start"),
                                       ctx.dev("q_len"), ctx.dev("pos0"), None, ctx.dev("seq_row"), table, None, None, 1,
                                       H, KV, HD, page, pages, self.window, self.scale, ctx.err,
-                                      rope=extra.get("rope"), cluster=plan["cluster"], keep=self.keep)
+                                      rope=extra.get("rope"), cluster=plan["cluster"], keep=self.keep,
+                                      sinks=extra.get("sinks"))
                 elif n_items:
                     flash(qkv, width, out, kpool, vpool, ctx.dev(form), n_items, decode, ctx.dev("q_start"),
                           ctx.dev("q_len"), ctx.dev("pos0"), ctx.dev(nm + "part_base"), ctx.dev("seq_row"),
@@ -399,20 +403,23 @@ class GatedAttention(PagedAttention):
     layer's values for the others, "mix" caches (1 - lam) v + lam v_kept, lam stored as `<vmix>`), a rotation of the first dims of a head (`position`, any rope spec), capped scores (`softcap`), a sink in
     the softmax's denominator (`sink`: "unit" -- a sink of score zero, so one is added to the denominator -- or the name
     of a tensor with one number per query head, or None) and a gate per token and query head (`gate`: head h's result
-    times sigmoid(Wg h)_h, Wg stored as `<g>`).  No biases.
+    times sigmoid(Wg h)_h, Wg stored as `<g>`).  `bias`: q, k and v have biases (the tensor's name with `.b`), added before anything
+    else happens to them.
 
         q = Wq h (heads x dim), k = Wk h (kv_heads x dim), v = Wv h (kv_heads x vdim)
         q, k <- rms(.) n per head;  rotated;  s = scale q . k, s <- cap tanh(s / cap)
         p_j = e^s_j / (e^sink + sum_j e^s_j);  out = Wo concat_h(sigmoid(g_h) sum_j p_j v_j)
 
-    One product makes q, k, v and the gates' logits; one kernel norms, rotates and writes k and v to their pages; the
-    attention kernel takes cap, sink and gate in.  Norms, angles, scores and the softmax are float32."""
+    One product makes q, k, v and the gates' logits; one kernel adds the biases, norms, rotates and writes k and v to
+    their pages (without norms and with equal widths a decode step leaves that to the attention kernel); the attention
+    kernel takes cap, sink and gate in.  Norms, angles, scores and the softmax are float32."""
 
     def __init__(self, hidden, heads, kv_heads, head_dim, vdim=None, scale=None, softcap=None, qk_norm=False, eps=1e-6,
-                 sink=None, gate=False, position=None, window=None, keep_first=0, value_mix=None, prefix="", names=None):
+                 sink=None, gate=False, position=None, window=None, keep_first=0, value_mix=None, bias=False, prefix="", names=None):
         super().__init__(heads, kv_heads, head_dim, window, scale, vdim=vdim, softcap=softcap, sinks=sink is not None,
                          gated=gate, keep_first=keep_first)
         self.D, self.eps, self.sink, self.gate = int(hidden), float(eps), sink, bool(gate)
+        self.has_bias, self.bias = bool(bias), None
         if qk_norm not in (True, False, None, "after") or value_mix not in (None, "keep", "mix"):
             raise ConfigError(f"this attention has no q/k norm {qk_norm!r} or value mixing {value_mix!r}")
         self.norm_at = "after" if qk_norm == "after" else ("before" if qk_norm else None)
@@ -432,6 +439,8 @@ class GatedAttention(PagedAttention):
         H, KV, HD, VD, D = self.H, self.KV, self.HD, self.VD, self.D
         out = [Want(self.n["q"], (H * HD, D), "matrix"), Want(self.n["k"], (KV * HD, D), "matrix"),
                Want(self.n["v"], (KV * VD, D), "matrix"), Want(self.n["o"], (D, H * VD), "matrix")]
+        if self.has_bias:
+            out += [Want(self.n[r] + ".b", (n,), "vector") for r, n in (("q", H * HD), ("k", KV * HD), ("v", KV * VD))]
         if self.value_mix == "mix":
             out.append(Want(self.n["vmix"], (), "vector"))
         if self.norm_at == "before":
@@ -450,6 +459,8 @@ class GatedAttention(PagedAttention):
         if rows % 8:        # rows of the product start on 16-byte boundaries in bfloat16: zero rows behind the gates
             parts.append(torch.zeros((8 - rows % 8, self.D), dtype=parts[0].dtype, device=parts[0].device))
         self.w_in = torch.cat(parts, 0).contiguous()
+        if self.has_bias:
+            self.bias = torch.cat([tensors[self.n[r] + ".b"] for r in "qkv"], 0).contiguous()
         self.wo = t("o")
         self.qw, self.kw = (t("q_norm"), t("k_norm")) if self.norm_at == "before" else (None, None)
         if self.value_mix == "mix":
@@ -481,17 +492,30 @@ class GatedAttention(PagedAttention):
         if self.position is not None:
             freqs, rd, pairing = self.position.rotation()
             gain = getattr(self.position, "gain", 1.0)
-        # the layer whose values others mix in runs first in the step and leaves them in a buffer of the step's tokens
-        kept = ctx.ws.get("values_kept", N, (KV * VD,), ctx.dtype) if self.value_mix else None
-        ops.norm_rope_kv_write(rows, self.qw, self.kw, self.eps, freqs, rd, pairing, gain, ctx.dev("positions"),
-                               ctx.dev("tok_row"), table, kpool if run.write else None, vpool if run.write else None, H, KV,
-                               HD, VD, page, pages, ctx.err, norm=self.norm_at,
-                               v_keep=kept if self.value_mix == "keep" else None,
-                               v_first=kept if self.value_mix == "mix" else None, lam=self.lam)
+        plain = self.norm_at is None and self.value_mix is None and HD == VD and not self.gate and gain == 1.0
+        # A step in which every sequence brings one token (N == S: that follows from the lengths of the step's arrays):
+        # the decode form of the TMA attention kernel adds the biases, rotates, stores and attends in one launch.
+        folded = (plain and run.write and N == ctx.S and not self.is_general(ctx) and self.uses_mma(ctx)
+                  and ctx.options.get("attention_kernel", "tma") == "tma" and ops.attention_tma_supports(HD, page)
+                  and ops.attention_tma_folds_rotation(H // KV) and ctx.options.get("attention_folds_rotation", True))
+        if folded:
+            pass
+        elif plain and rows.shape[1] == (H + 2 * KV) * HD and freqs is not None:
+            ops.rope_kv_write(rows, self.bias, ctx.dev("positions"), ctx.dev("tok_row"), table, kpool if run.write else None,
+                              vpool if run.write else None, freqs, H, KV, HD, rd, pairing, page, pages, ctx.err)
+        else:
+            # the layer whose values others mix in runs first in the step and leaves them in a buffer of the step's tokens
+            kept = ctx.ws.get("values_kept", N, (KV * VD,), ctx.dtype) if self.value_mix else None
+            ops.norm_rope_kv_write(rows, self.qw, self.kw, self.eps, freqs, rd, pairing, gain, ctx.dev("positions"),
+                                   ctx.dev("tok_row"), table, kpool if run.write else None, vpool if run.write else None, H,
+                                   KV, HD, VD, page, pages, ctx.err, norm=self.norm_at,
+                                   v_keep=kept if self.value_mix == "keep" else None,
+                                   v_first=kept if self.value_mix == "mix" else None, lam=self.lam, bias=self.bias)
         o = ctx.ws.get("gattn_out", N, (H * VD,), ctx.dtype)
         off = (H + KV) * HD + KV * VD
         gate = rows[:, off:off + H] if self.gate else None
-        self.attend(ctx, rows, rows.stride(0), o, table, kpool, vpool, sinks=self.sinks, gate=gate)
+        self.attend(ctx, rows, rows.stride(0), o, table, kpool, vpool, sinks=self.sinks, gate=gate,
+                    rope=(self.bias, freqs, rd, pairing) if folded else None)
         y = ctx.ws.get(out, N, (self.D,), ctx.dtype)
         ops.linear(o, self.wo, out=y)
         return y, None

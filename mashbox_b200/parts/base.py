@@ -74,11 +74,13 @@ class LayerRun:
     with the cache id its entry gives) and an entry may read a cache another layer wrote (write=False).  Fixed-size
     state of the run (what its parts carry from step to step besides the cache) is kept under `state`; None: under
     the cache id, as a run that owns its cache wants it.  A run that borrows a cache but carries state of its own
-    names an id no other run has."""
+    names an id no other run has.  `rejoin`: the embedding's output (the stream as the first run found it) is added into the
+    stream right before this run."""
     layer: int
     cache: int = None
     write: bool = True
     state: int = None
+    rejoin: bool = False
 
     @property
     def state_id(self):
@@ -240,6 +242,14 @@ class StepContext:
     # it runs a part; the model names the first norm of the block that runs next in `next_first_norm`.
     after_norm = None
     next_first_norm = None
+
+    # What joins the stream after the block that runs now, besides its own output: (N, D) float32 rows, or None.  A block
+    # that adds them in a kernel of its own takes them (take_joining); the model adds what is left.
+    joining = None
+
+    def take_joining(self):
+        j, self.joining = self.joining, None
+        return j
 
     def add_into_stream(self, a, w, x, bias=None):
         """x (N, D) float32 += a W^T (+ bias), in place"""

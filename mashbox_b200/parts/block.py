@@ -220,7 +220,8 @@ class SandwichBlock:
     the normed outputs channel by channel and are multiplied into the post norms' weights at load.  One kernel norms a
     sublayer's output, adds it into the float32 stream and makes the norm that reads the stream next -- the
     feed-forward's pre norm, or the first norm of the block that runs next -- so the stream is read once per sublayer.
-    `ffn` may be None (the layer has no feed-forward), `side` may be None.  Nothing is left pending."""
+    What joins the stream after the block (ctx.joining) is added by the same kernel.  `ffn` may be None (the layer has no
+    feed-forward), `side` may be None.  Nothing is left pending."""
     graph_safe = True       # forward() depends on the batch only through the lengths of the step's arrays
 
     def __init__(self, prefix, mixer, norm, ffn=None, side=None, scale1=None, scale2=None, names=None):
@@ -281,12 +282,13 @@ class SandwichBlock:
             if bias is not None:
                 raise ConfigError("a sandwich block cannot norm an output with a deferred bias")
             last = i == len(steps) - 1
+            again = ctx.take_joining() if last and self.side is None else None
             follow = (self.pre2 if not last else (nxt if self.side is None else None))
             h = ctx.ws.get("normed", x.shape[0], (self.width,), ctx.dtype) if follow is not None else None
             if last and self.side is not None and ctx.dtype != torch.float32:
                 xa = ctx.ws.get("stream_copy", x.shape[0], (self.width,), ctx.dtype)
             ops.post_norm_add(x, y, w, post.eps, follow.weight if follow is not None else None,
-                              follow.eps if follow is not None else 0.0, h, xa)
+                              follow.eps if follow is not None else 0.0, h, xa, again=again)
         if self.side is not None:
             h = ctx.ws.get("normed", x.shape[0], (self.width,), ctx.dtype) if nxt is not None else None
             self.side.forward(ctx, x, x if xa is None else xa, nxt, h)

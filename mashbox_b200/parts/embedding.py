@@ -69,10 +69,12 @@ class NormedEmbedding(Embedding):
 
 class LinearHead:
     graph_safe = True       # forward() depends on the batch only through the lengths of the step's arrays
-    def __init__(self, vocab, hidden, tied, name="output.weight", tied_to="token_embd.weight", scale=1.0):
-        """scale: the logits are multiplied by it (in float32, after the product)"""
+    def __init__(self, vocab, hidden, tied, name="output.weight", tied_to="token_embd.weight", scale=1.0,
+                 softcap=None):
+        """scale: the logits are multiplied by it (in float32, after the product); softcap: they become
+        softcap tanh(l / softcap) after that"""
         self.V, self.D, self.tied, self.name, self.tied_to = int(vocab), int(hidden), bool(tied), name, tied_to
-        self.scale = float(scale)
+        self.scale, self.softcap = float(scale), float(softcap) if softcap else None
         self.weight = None
 
     def wants(self):
@@ -87,6 +89,8 @@ class LinearHead:
         ctx.ops.linear(h, self.weight, out=out, out_dtype=torch.float32)
         if self.scale != 1.0:
             ctx.ops.scale_rows(out, self.scale)
+        if self.softcap is not None:
+            ctx.ops.softcap_rows(out, self.softcap)
         return out
 
 

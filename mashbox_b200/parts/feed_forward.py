@@ -1,5 +1,5 @@
-"""Dense SwiGLU feed-forward: (silu(h Wg^T) * (h Wu^T)) Wd^T, silu and the product in float32
-(src/mashbox/gguf/archs/dense.py:356-357).  Gate and up weights are concatenated at load so one product makes both."""
+"""Dense gated feed-forward: (act(h Wg^T) * (h Wu^T)) Wd^T, act silu (SwiGLU, src/mashbox/gguf/archs/dense.py:356-357) or
+the tanh form of gelu, act and the product in float32.  Gate and up weights are concatenated at load so one product makes both."""
 import math
 
 from ..weights.loader import Want
@@ -8,6 +8,8 @@ from .base import register
 
 class SwiGLU:
     graph_safe = True       # forward() depends on the batch only through the lengths of the step's arrays
+    MODE = "swiglu"         # the name of the gate in the kernels' faces
+
     def __init__(self, hidden, intermediate, prefix="", names=None):
         self.D, self.F = int(hidden), int(intermediate)
         n = dict(gate="ffn_gate", up="ffn_up", down="ffn_down")
@@ -37,11 +39,11 @@ class SwiGLU:
             w, eps = norm.fusable()
             ctx.ops.linear_small_normed(x, w, eps, self.wgu, a, "swiglu", held=ctx.take_held(x, norm))
         elif ctx.dtype == torch.bfloat16 and ctx.ops.fused_swiglu_supports(N, self.F, self.D):
-            ctx.ops.linear_swiglu(h, self.wgu, a)           # both products and the gate in one kernel
+            ctx.ops.linear_swiglu(h, self.wgu, a, self.MODE)        # both products and the gate in one kernel
         else:
             gu = ctx.ws.get("gate_up", N, (2 * self.F,), ctx.dtype)
             ctx.ops.linear(h, self.wgu, out=gu)
-            ctx.ops.swiglu(gu, a)
+            getattr(ctx.ops, self.MODE)(gu, a)
         if residual is not None:
             ctx.add_into_stream(a, self.wd, residual)
             return None
@@ -51,6 +53,15 @@ class SwiGLU:
 
 
 register("feed_forward", "swiglu", SwiGLU)
+
+
+class GeGLU(SwiGLU):
+    """the same unit with gelu_tanh(z) = z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) on the gate"""
+    MODE = "geglu"
+    fuses_small = False     # the products of a normed stream have silu's gate only
+
+
+register("feed_forward", "geglu", GeGLU)
 
 
 def _softplus(t):

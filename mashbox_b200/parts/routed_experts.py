@@ -11,7 +11,9 @@ expert (`router_bias`: its tensor), which counts in choice and weights alike; a 
 worth its largest c alone (`group_worth="max"`); the weights may be multiplied by a constant (`scale`); the expert may be
 the plain gated form Wd (silu(Wg h) * (Wu h)) (`limit=None, alpha=1, shift=0`: no clamps, nothing added to u); and an
 expert that every token uses (`shared`: the spec of a feed-forward part, its tensors under `shared_prefix`) may be added,
-times sigmoid(w_sg . h) when `shared_gate` names such a row (its logit is one more row of the router's product).
+times sigmoid(w_sg . h) when `shared_gate` names such a row (its logit is one more row of the router's product).  A weight
+may meet the expert's input instead of its output (`weigh="input"`): out = sum of expert_e(s_e h), where the gate and up
+products, linear in their input, are multiplied by s_e in the kernel that makes them.
 
 The correction moves the choice only: the weights are the plain scores, not renormalised.  The stored matrices of the
 experts (`e0`, `e1`, ...) are stacked at load into (experts, rows, columns) tensors.  A step: the router's product with
@@ -32,13 +34,16 @@ class RoutedExperts:
 
     def __init__(self, hidden, intermediate, experts, top, limit, groups=1, keep=1, alpha=1.702, correction=True,
                  score="sigmoid", group_worth="top2", scale=1.0, shift=1.0, shared=None, shared_prefix="mlp.shared.",
-                 shared_gate=None, router_bias=None, prefix="", names=None):
+                 shared_gate=None, router_bias=None, weigh="output", prefix="", names=None):
         self.D, self.F, self.E, self.top = int(hidden), int(intermediate), int(experts), int(top)
         self.groups, self.keep = int(groups or 1), int(keep or 1)
         self.limit = float(limit) if limit is not None else float("inf")
         self.alpha, self.has_correction = float(alpha), bool(correction)
         if score not in ("sigmoid", "softmax", "softmax_chosen") or group_worth not in ("top2", "max"):
             raise ConfigError(f"routed experts: score {score!r} / group worth {group_worth!r} are not known")
+        if weigh not in ("output", "input"):
+            raise ConfigError(f"routed experts: a weight meets an expert's output or its input, not {weigh!r}")
+        self.weigh_input = weigh == "input"
         self.score, self.group_worth, self.scale, self.shift = score, group_worth, float(scale), float(shift)
         self.shared = make("feed_forward", shared, prefix=prefix + shared_prefix) if shared is not None else None
         self.shared_gate = prefix + shared_gate if (shared_gate and self.shared is not None) else None
@@ -110,21 +115,25 @@ class RoutedExperts:
             scratch = ctx.ws.get("expert_places", ctx.ws.max_rows * self.top + T, (), torch.int32,
                                  reserve=ctx.ws.max_rows * self.top + T)
             delta = ctx.ws.get(out, N, (self.D,), ctx.dtype)
-            ops.moe_tc5(h, ids, wts, self.wgu, self.wd, delta, rows, act, y, scratch, self.limit, self.alpha, self.shift, ys, gate)
+            scale = ctx.ws.get("expert_row_scale", 128 * T, (), torch.float32, reserve=128 * T) if self.weigh_input else None
+            ops.moe_tc5(h, ids, wts, self.wgu, self.wd, delta, rows, act, y, scratch, self.limit, self.alpha, self.shift, ys,
+                        gate, row_scale=scale)
             return delta, None
         y = ctx.ws.get("expert_out", N, (self.top, self.D), torch.float32)
+        in_wts, out_wts = (wts, None) if self.weigh_input else (None, wts)
         if ops.moe_grouped_supports(N, self.D, self.F, ctx.dtype) and not ctx.options.get("plain_experts", False):
             act = ctx.ws.get("expert_act", N * self.top, (self.F,), ctx.dtype, reserve=ctx.ws.max_rows * self.top)
             n = ops.moe_grouped_scratch(ctx.ws.max_rows, self.top, self.E)
             scratch = ctx.ws.get("expert_sort", max(n, ops.moe_grouped_scratch(N, self.top, self.E)), (), torch.int32, reserve=n)
-            ops.moe_grouped(h, ids, self.wg, self.wu, self.wd, y, act, scratch, self.limit, self.alpha, self.shift)
+            ops.moe_grouped(h, ids, self.wg, self.wu, self.wd, y, act, scratch, self.limit, self.alpha, self.shift,
+                            in_wts)
         else:
             # bfloat16 steps of many tokens take the other form: room for the few
             most = min(ctx.ws.max_rows, max(N, ops.MOE_GROUPED["tokens"])) if ctx.dtype == torch.bfloat16 else ctx.ws.max_rows
             act = ctx.ws.get("expert_act_few", N * self.top, (self.F,), torch.float32, reserve=most * self.top)
-            ops.moe_experts(h, ids, self.wg, self.wu, self.wd, y, self.limit, self.alpha, act, self.shift)
+            ops.moe_experts(h, ids, self.wg, self.wu, self.wd, y, self.limit, self.alpha, act, self.shift, in_wts)
         delta = ctx.ws.get(out, N, (self.D,), ctx.dtype)
-        ops.moe_combine(y, wts, delta, ys, gate)
+        ops.moe_combine(y, out_wts, delta, ys, gate)
         return delta, None
 
 

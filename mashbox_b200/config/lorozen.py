@@ -131,8 +131,8 @@ class LorozenConfig:
             return Rotation(dims=dims, base=float(need(rot, "base", w + "rot.")), scaling=scaling)
 
         def window(m, w):
-            mask = m.get("mask") or None
-            if not mask:
+            mask = m.get("mask")
+            if mask is None:
                 return None
             size = int(need(mask, "size", w + "mask."))
             if size < 1:

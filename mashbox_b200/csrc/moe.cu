@@ -70,9 +70,11 @@ __global__ void moe_select_kernel(const float* __restrict__ z, int z_stride, con
         }
     } else {
         for (int e = lane; e < E; e += 32) {
-            const float v = 1.0f / (1.0f + expf(-logit(e)));
+            const float z1 = logit(e), v = 1.0f / (1.0f + expf(-z1));
             s[e] = v;
-            c[e] = v + (correction ? correction[e] : 0.0f);
+            // without a correction and without groups the logits order the experts as their scores do, also where the scores
+            // round to one
+            c[e] = correction ? v + correction[e] : groups > 1 ? v : z1;
         }
     }
     __syncwarp();

@@ -940,6 +940,230 @@ def pobelorn_kernels(a, z, P, B, ctx, pk):
     return res
 
 
+# Layer sizes for `--design lorozen`: attention (a window of 4,096 positions, heads of 128 x 128 of which half a head is
+# rotated, a kv head to four query heads, biases and sinks) first, wkv (heads of 128) twice, latent attention last (latents of
+# 128 values with a rotated strip of 64, a window of 4,096, a gate per head); a dense unit in the first layer, routed experts
+# weighted at their input beside a shared one in the others; no loop.  The Sufopel decoder beside it -- the closest design the
+# engine has: sandwich blocks, a recurrence with a matrix state per head and a decay per key channel, latent attention every
+# fourth layer, routed experts -- has the same width, layers, heads, head sizes and as many active expert weights, and no
+# token input.
+LOROZEN_SIZES = {k: dict(width=v["width"], heads=v["heads"], dim=128, kv_rank=128, rot=64, window=4096, ff=v["ff"], experts=64,
+                         top=v["top"] - 1, groups=8, keep=4, q_rank=v["q_rank"], rank=64) for k, v in SUFOPEL_SIZES.items()}
+
+
+def lorozen_configs(size, layers, vocab=32000, context=8192):
+    from mashbox_b200.config import lorozen as F
+    from mashbox_b200.config.sufopel import DeltaMixer, DenseFF, LatentMixer, RoutedFF, SufopelConfig, SufopelLayer
+    z = LOROZEN_SIZES[size]
+    D, H, dim, top = z["width"], z["heads"], z["dim"], z["top"] + 1
+    att = F.AttentionMixer(heads=H, kv_heads=max(1, H // 4), dim=dim, vdim=dim, scale=dim ** -0.5, window=z["window"],
+                           rot=F.Rotation(dim // 2, 500000.0, (8.0, 1.0, 4.0, 4096.0)))
+    wkv = F.WkvMixer(heads=H, dim=dim, decay_rank=z["rank"])
+    lat = F.LatentMixer(heads=H, dim=dim, vdim=dim, kv_rank=z["kv_rank"], scale=(dim + z["rot"]) ** -0.5, rot_dim=z["rot"],
+                        rot=F.Rotation(z["rot"], 500000.0), window=z["window"])
+    kinds = (("attention", att), ("wkv", wkv), ("wkv", wkv), ("latent_attention", lat))
+    moe = F.ExpertsFF(ff=z["ff"], experts=z["experts"], top=z["top"], shared_ff=z["ff"])
+    lz = F.LorozenConfig("Lorozen", width=D, vocab=vocab, norm_eps=1e-6, logit_softcap=30.0, layers=tuple(
+        F.LorozenLayer(*kinds[i % 4], F.DenseFF(z["ff"] * top) if i == 0 else moe) for i in range(layers)))
+    dl = DeltaMixer(heads=H, kv_heads=H, dim=dim, vdim=dim, conv=4, a_rank=z["rank"], g_rank=z["rank"])
+    la = LatentMixer(heads=H, dim=dim, vdim=dim, q_rank=z["q_rank"], kv_rank=z["kv_rank"], scale=dim ** -0.5)
+    rt = RoutedFF(ff=z["ff"], limit=7.0, experts=z["experts"], top=top, groups=z["groups"], keep=z["keep"])
+    sf = SufopelConfig("Sufopel", width=D, vocab=vocab, max_positions=context + 2048, embedding_scale=1.0, logit_scale=1.0,
+                       norm_eps=1e-6, side_dim=None, layers=tuple(
+        SufopelLayer("latent_attention" if i % 4 == 3 else "channel_delta", la if i % 4 == 3 else dl,
+                     DenseFF(z["ff"] * top) if i == 0 else rt) for i in range(layers)))
+    return lz, sf
+
+
+def lorozen_kernels(a, z, P, B, ctx, pk):
+    """The kernels of the Lorozen decoder, each beside the like kernel of the Sufopel (or Llama, or Fipitar) decoder at
+    equal sizes: CUDA-event time of single launches after an L2 flush, and the fraction of the measured peak that the
+    algorithmic bytes (copy bandwidth) or FLOPs (bf16 tensor throughput) come to."""
+    import torch
+    from mashbox_b200 import ops
+    from mashbox_b200.parts.attention import PagedAttention
+    dev = "cuda:0"
+    D, H, dim, R, rd, F, E, top = (z[k] for k in ("width", "heads", "dim", "kv_rank", "rot", "ff", "experts", "top"))
+    page, win, KV, C, rank = 16, z["window"], max(1, H // 4), H * dim, z["rank"]
+    gen = torch.Generator(device=dev).manual_seed(0)
+    bf = lambda *s: (torch.randn(*s, generator=gen, device=dev) * 0.5).to(torch.bfloat16)
+    f32 = lambda *s: torch.randn(*s, generator=gen, device=dev) * 0.5
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    err = ops.new_error_word(dev)
+
+    def timed(f):
+        for _ in range(3):
+            f()
+        ts = []
+        for _ in range(max(5, a.steps // 4)):
+            flush.zero_()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            f()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) * 1e3)
+        return statistics.median(ts)
+
+    mem = lambda us, nbytes: {"us": us, "gbs": nbytes / us / 1e3, "frac_of_copy_peak": nbytes / us / 1e3 / pk["hbm_gbs"]}
+    mat = lambda us, flops: {"us": us, "tflops": flops / us / 1e6, "frac_of_bf16_peak": flops / us / 1e6 / pk["bf16_tflops"]}
+    res = {}
+    # ---- wkv: the recurrence beside the delta rule and the gated scan of equal size; what stands around it
+    for form, N, S in (("prompt", P, 1), ("decode", B, B)):
+        n = N // S
+        seq = (i32([i * n for i in range(S)]), i32([n] * S), i32(list(range(S))))
+        tok_seq = i32([i // n for i in range(N)])
+        r, k, v, o = (f32(N, C) for _ in range(4))
+        g, share = torch.rand(N, C, generator=gen, device=dev), f32(N, H)
+        state = torch.zeros(S, D + C * dim, device=dev)
+        sv = state[:, D:]
+        nbytes = 2 * S * C * dim * 4 + N * C * 5 * 4
+        us = timed(lambda: ops.gated_scan(r, k, v, g, o, sv, seq, H, H, dim, dim, False, bonus=share))
+        res[f"wkv_scan_{form}"] = mem(us, nbytes)
+        us = timed(lambda: ops.gated_scan(r, k, v, g, o, sv, seq, H, H, dim, dim, False))
+        res[f"gla_scan_fipitar_{form}"] = mem(us, nbytes)
+        us = timed(lambda: ops.delta_rule(r, k, v, g, share, o, sv, seq, H, H, dim, dim))
+        res[f"delta_rule_sufopel_{form}"] = mem(us, nbytes)
+        h, mu, mixes = bf(N, D), torch.rand(5, D, generator=gen, device=dev), torch.empty(5, N, D, device=dev, dtype=torch.bfloat16)
+        us = timed(lambda: ops.token_mix(h, mu, state[:, :D], (tok_seq,) + seq, mixes))
+        res[f"token_mix_{form}"] = mem(us, N * D * 2 * 6)
+        cw, cs, cy = f32(4, 3 * C), torch.zeros(S, 9 * C, device=dev), torch.empty(N, 3 * C, device=dev, dtype=torch.bfloat16)
+        cx = bf(N, 3 * C)
+        us = timed(lambda: ops.short_conv(cx, cw, cs, (tok_seq,) + seq, cy))
+        res[f"short_conv_sufopel_{form}"] = mem(us, N * 3 * C * 4)
+        w4, rows = bf(4 * C, D), torch.empty(N, 4 * C, device=dev, dtype=torch.bfloat16)
+        us = timed(lambda: ops.linear_groups(mixes[:4], w4, rows))
+        us1 = timed(lambda: ops.linear(h, w4, out=rows))
+        if form == "prompt":
+            res["four_products_prompt"], res["one_product_as_large_prompt"] = mat(us, 8 * N * C * D), mat(us1, 8 * N * C * D)
+        else:
+            res["four_products_decode"], res["one_product_as_large_decode"] = mem(us, 8 * C * D), mem(us1, 8 * C * D)
+        rows = bf(N, 4 * C)
+        w0, u, zz, low, w2 = f32(C), f32(C), f32(N, C), f32(N, rank), bf(C, rank)
+        if form == "prompt":
+            us = timed(lambda: ops.wkv_gates(rows, w0, u, r, k, v, g, share, H, dim, z=zz))
+            res["wkv_gates_prompt"] = mem(us, N * C * (3 * 2 + 4 + 4 * 4))
+        else:
+            us = timed(lambda: ops.wkv_gates(rows, w0, u, r, k, v, g, share, H, dim, low=low, w2=w2))
+            res["wkv_gates_with_product_decode"] = mem(us, C * rank * 2 + N * C * (3 * 2 + 4 * 4))
+        us = timed(lambda: ops.gla_gates(rows, zz, w0, 16.0, r, k, v, g, H, dim, dim))
+        res[f"gla_gates_fipitar_{form}"] = mem(us, N * C * (3 * 2 + 4 + 4 * 4))
+        gated, nw = torch.empty(N, C, device=dev, dtype=torch.bfloat16), f32(H, dim)
+        us = timed(lambda: ops.gated_rms(o, rows[:, 3 * C:], nw, gated, H, dim, 1e-6, silu=True))
+        res[f"wkv_norm_gate_{form}"] = mem(us, N * C * (4 + 2 + 2))
+        us = timed(lambda: ops.gated_rms(o, rows[:, 3 * C:], nw[0], gated, H, dim, 1e-6))
+        res[f"delta_norm_gate_sufopel_{form}"] = mem(us, N * C * (4 + 2 + 2))
+        del state, w4
+    # ---- attention: a prompt of P tokens; a portion of P tokens far behind the window; B tokens decoded at ctx.  With a sink
+    #      beside Llama's over as many keys; with values half as wide, on the general kernel, beside Fipitar's; latents with a
+    #      window and a gate beside Fipitar's with a sink
+    own, llama = PagedAttention(H, KV, dim, win, sinks=True), PagedAttention(H, KV, dim)
+    narrow = PagedAttention(H, KV, dim, win, vdim=dim // 2, sinks=True)
+    fip = PagedAttention(H, KV, dim, None, vdim=dim // 2, softcap=30.0, sinks=True)
+    lat = PagedAttention(H, 1, R + rd, win, (dim + rd) ** -0.5, vdim=R, gated=True)
+    flat = PagedAttention(H, 1, R + rd, None, (dim + rd) ** -0.5, vdim=R, sinks=True)
+    sinks = f32(H)
+    for name, core, wk, wv in (("attention", own, dim, dim), ("attention_llama", llama, dim, dim),
+                               ("attention_narrow_values", narrow, dim, dim // 2), ("attention_fipitar", fip, dim, dim // 2),
+                               ("latent_attention", lat, R + rd, R), ("latent_attention_fipitar", flat, R + rd, R)):
+        one_row = core in (lat, flat)
+        for form, N, S, end in (("prompt", P, 1, P), ("portion", P, 1, max(ctx, win + P)), ("decode", B, B, ctx)):
+            pairs = min(win, ctx)               # keys a query sees far from the start; the others are given as many
+            if form != "prompt" and not core.window:
+                end = pairs if form == "decode" else pairs + P // 2
+            pages = S * -(-end // page)
+            table = torch.arange(pages, dtype=torch.int32, device=dev).reshape(S, -1)
+            kp = bf(pages, core.KV, page, wk)
+            vp = kp if one_row else bf(pages, core.KV, page, wv)
+            q, o = bf(N, H * wk), torch.empty(N, H * wv, device=dev, dtype=torch.bfloat16)
+            q_len = [N // S] * S
+            ctx_ = _PlanContext(ops, dev, q_len, [end - n for n in q_len], page, pages, err)
+            core.prepare(ctx_)
+            ctx_.inputs.upload()
+            extra = dict(sinks=sinks) if core.sunk else {}
+            if core is lat:
+                extra["gate"] = bf(N, H)
+            us = timed(lambda: core.attend(ctx_, q, H * wk, o, table, kp, vp, **extra))
+            if form == "decode":
+                res[f"{name}_{form}"] = mem(us, S * pairs * core.KV * (wk + (0 if one_row else wv)) * 2 + N * H * (wk + wv) * 2)
+            else:
+                res[f"{name}_{form}"] = mat(us, 2 * H * (wk + wv) * P * (P / 2 if form == "prompt" else pairs))
+            del kp, vp
+    # ---- heads between the product and attention (biases, rotation, cache write); Llama's without biases
+    for form, N in (("prompt", P), ("decode", B)):
+        rows = bf(N, (H + 2 * KV) * dim)
+        pages = -(-N // page)
+        table = torch.arange(pages, dtype=torch.int32, device=dev).reshape(1, -1)
+        kp, vp, bias = bf(pages, KV, page, dim), bf(pages, KV, page, dim), f32((H + 2 * KV) * dim)
+        pos, row = torch.arange(N, dtype=torch.int32, device=dev), torch.zeros(N, dtype=torch.int32, device=dev)
+        fr = torch.rand(dim // 2, generator=gen, device=dev)
+        nbytes = 2 * N * (H + 2 * KV) * dim * 2
+        for name, b in (("heads", bias), ("heads_llama", None)):
+            us = timed(lambda: ops.rope_kv_write(rows, b, pos, row, table, kp, vp, fr, H, KV, dim, dim // 2, 1, page, pages, err))
+            res[f"{name}_{form}"] = mem(us, nbytes)
+        us = timed(lambda: ops.norm_rope_kv_write(rows, None, None, 1e-6, fr, dim // 2, 1, 1.0, pos, row, table, kp, vp, H, KV, dim,
+                                                  dim, page, pages, err, norm=None, bias=bias))
+        res[f"heads_unequal_widths_{form}"] = mem(us, nbytes)
+        qw = f32(dim)
+        us = timed(lambda: ops.norm_rope_kv_write(rows, qw, qw, 1e-6, fr, dim // 2, 1, 1.0, pos, row, table, kp, vp, H, KV, dim,
+                                                  dim, page, pages, err))
+        res[f"heads_fipitar_{form}"] = mem(us, nbytes)
+    # ---- the experts weighted at their input, and at their output (Sufopel's); the dense unit's two gates
+    wg, wu, wd = bf(E, F, D), bf(E, F, D), bf(E, D, F)
+    Fd = F * (top + 1)
+    for form, N in (("prompt", P), ("decode", B)):
+        h = bf(N, D)
+        ids = torch.stack([torch.randperm(E, generator=gen, device=dev)[:top] for _ in range(N)]).int().contiguous()
+        wts, shared = torch.rand(N, top, generator=gen, device=dev), bf(N, D)
+        touched = len(set(ids.flatten().tolist()))
+        out = torch.empty(N, D, device=dev, dtype=torch.bfloat16)
+        for name, own_ in (("experts", True), ("experts_sufopel", False)):
+            if form == "prompt":
+                T = ops.moe_tc5_tiles(N, top, E)
+                rows, act2 = torch.empty(128 * T, D, device=dev, dtype=torch.bfloat16), torch.empty(128 * T, F, device=dev, dtype=torch.bfloat16)
+                y2, places = torch.empty(128 * T, D, device=dev), torch.empty(N * top + T, dtype=torch.int32, device=dev)
+                scale = torch.empty(128 * T, device=dev) if own_ else None
+                wgu2 = torch.cat([wg, wu], 1).contiguous()
+                us = timed(lambda: ops.moe_tc5(h, ids, wts, wgu2, wd, out, rows, act2, y2, places, float("inf"), 1.0, 0.0, shared,
+                                               None, row_scale=scale))
+                res[f"{name}_prompt"] = mat(us, 2 * N * top * 3 * F * D)
+                need = max(2 * N * top * 3 * F * D / (pk["bf16_tflops"] * 1e6), touched * 3 * F * D * 2 / (pk["hbm_gbs"] * 1e3))
+                res[f"{name}_prompt"].update(frac_of_roofline=need / us)
+                del wgu2, rows, act2, y2
+            else:
+                y = torch.empty(N, top, D, device=dev)
+                us = timed(lambda: (ops.moe_experts(h, ids, wg, wu, wd, y, float("inf"), 1.0, None, 0.0, wts if own_ else None),
+                                    ops.moe_combine(y, None if own_ else wts, out, shared)))
+                res[f"{name}_decode"] = dict(mem(us, touched * 3 * F * D * 2), experts_touched=touched)
+        zl, corr = f32(N, E), f32(E)
+        idc, wtc = torch.empty(N, top, dtype=torch.int32, device=dev), torch.empty(N, top, device=dev)
+        res[f"choice_{form}"] = {"us": timed(lambda: ops.moe_select(zl, None, idc, wtc, experts=E))}
+        res[f"choice_sufopel_{form}"] = {"us": timed(lambda: ops.moe_select(zl, corr, idc, wtc, z["groups"], z["keep"], experts=E))}
+        wgu, wdn, a1 = bf(2 * Fd, D), bf(D, Fd), torch.empty(N, Fd, device=dev, dtype=torch.bfloat16)
+        for name, mode in (("dense", "geglu"), ("dense_llama", "swiglu")):
+            if form == "prompt":
+                us = timed(lambda: ops.linear_swiglu(h, wgu, a1, mode))
+                res[f"{name}_gate_up_prompt"] = mat(us, 2 * N * 2 * Fd * D)
+            else:
+                us = timed(lambda: (ops.linear_swiglu(h, wgu, a1, mode) if ops.fused_swiglu_supports(N, Fd, D) else
+                                    ops.linear_stream(h, wgu, a1, mode), ops.linear(a1, wdn, out=out)))
+                res[f"{name}_decode"] = mem(us, 3 * Fd * D * 2)
+        del wgu, wdn
+    # ---- the stream: the norm of an output with the embedding joining, without (Sufopel's); the cap on the logits
+    for form, N in (("prompt", P), ("decode", B)):
+        x, d1, w, e = f32(N, D), bf(N, D), f32(D), f32(N, D)
+        nrm = torch.empty(N, D, device=dev, dtype=torch.bfloat16)
+        us = timed(lambda: ops.post_norm_add(x, d1, w, 1e-6, w, 1e-6, nrm, again=e))
+        res[f"post_norm_add_joined_{form}"] = mem(us, N * D * (4 + 4 + 2 + 2 + 4))
+        us = timed(lambda: ops.post_norm_add(x, d1, w, 1e-6, w, 1e-6, nrm))
+        res[f"post_norm_add_sufopel_{form}"] = mem(us, N * D * (4 + 4 + 2 + 2))
+    lg = f32(B, 32000)
+    res["softcap_decode"] = mem(timed(lambda: ops.softcap_rows(lg, 30.0)), B * 32000 * 8)
+    res["scale_rows_sufopel_decode"] = mem(timed(lambda: ops.scale_rows(lg, 1.0)), B * 32000 * 8)
+    return res
+
+
 def fipitar_kernels(a, z, P, B, ctx, pk):
     """The kernels of the Fipitar decoder, each beside the like kernel of the Sufopel (or Llama) decoder at equal sizes:
     CUDA-event time of single launches after an L2 flush, and the fraction of the measured peak that the algorithmic bytes
@@ -1082,7 +1306,11 @@ def run_design(a):
     layers = a.layers or 4
     design = a.design
     other = "llama"
-    if design == "pobelorn":
+    if design == "lorozen":
+        z, other = LOROZEN_SIZES[a.size], "sufopel"
+        cfgs = dict(zip((design, other), lorozen_configs(a.size, layers, context=a.context)))
+        single_kernels = lorozen_kernels
+    elif design == "pobelorn":
         z, other = POBELORN_SIZES[a.size], "tosevik"
         cfgs = dict(zip((design, other), pobelorn_configs(a.size, layers, context=a.context)))
         single_kernels = pobelorn_kernels
@@ -1638,8 +1866,8 @@ def main():
     ap.add_argument("--requests", type=int, default=0, help="workloads: fewer requests than the workload names")
     ap.add_argument("--pool-tokens", type=int, default=0, help="workloads: size of the cache pool (0: every request fits)")
     ap.add_argument("--seed", type=int, default=0)
-    ap.add_argument("--design", default="", choices=("", "luzosun", "sufopel", "tosevik", "fipitar", "pobelorn"),
-                    help="another design beside the Llama decoder of equal size (tosevik and fipitar: beside the Sufopel decoder, "
+    ap.add_argument("--design", default="", choices=("", "luzosun", "sufopel", "tosevik", "fipitar", "pobelorn", "lorozen"),
+                    help="another design beside the Llama decoder of equal size (tosevik, fipitar and lorozen: beside the Sufopel decoder, "
                     "pobelorn: beside the Tosevik decoder): "
                     "prefill, decode, single kernels")
     ap.add_argument("--size", default="8b", choices=tuple(DESIGN_SIZES), help="--design: the layer sizes")

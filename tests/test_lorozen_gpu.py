@@ -702,6 +702,25 @@ def test_windows_free_pages_for_a_pool_smaller_than_the_sequence(tmp_path_factor
     runner.cache.check()
 
 
+@pytest.mark.parametrize("name", ["P", "S"])
+def test_the_embedding_joins_behind_a_block_that_does_not_take_it_in(tmp_path_factory, monkeypatch, name):
+    """a block that leaves what joins the stream to the model, after it has made the next norm's output already"""
+    from mashbox_b200.parts.block import SandwichBlock
+    own = SandwichBlock.forward
+
+    def forward(self, ctx, x, pending, run):
+        rows = ctx.take_joining()
+        pending = own(self, ctx, x, pending, run)
+        ctx.joining = rows
+        return pending
+    monkeypatch.setattr(SandwichBlock, "forward", forward)
+    for dtype in DTYPES:
+        folder, runner = runner_for(tmp_path_factory.mktemp("m"), name, dtype, 128)
+        (p,) = S.prompts_for(name, (60,), seed=9)
+        got = joined(replay(runner, cut_steps("a", p, [30, 2] + [1] * 28)))
+        S.assert_close(got, S.plain_logits(folder, p), dtype, f"{name}: joined by the model")
+
+
 @pytest.mark.parametrize("name,dtype", [("P", "float32"), ("Q", "float32"), ("R", "bfloat16"), ("S", "float32")])
 def test_greedy_generation_through_the_engine(tmp_path_factory, name, dtype):
     """Engine.generate with its scheduler, graphs and sampler: three prompts of unequal length in portions of at most

@@ -25,7 +25,7 @@
 // Forms (EPI): 0 bf16 out; 1 SwiGLU (W = [gate rows | up rows], out = silu(gate) * up); 2 float out; 3 the float32
 // residual stream is added to in place (+ bias), and on request the product leaves what the norm after it needs: the
 // sums of squares of the new rows by 32 columns and the new rows times that norm's weight, in bf16; 4 bf16 out, the
-// square of the product's positive part; 5 as 1 with the tanh form of gelu.  (Rotation and the
+// square of the product's positive part; 5 as 1 with the tanh form of gelu; 6 as 0 with an input per group of rows of W.  (Rotation and the
 // cache write stay a kernel of their own after the q/k/v product: as an epilogue here, sixteen values per thread on
 // the few warps that finish a tile, they cost 9 to 15 us against its 3.)  SCALED: the input is such a pair (rows
 // times the norm's weight in bf16, sums of squares): the token's 1/rms, computed in float from the sums, scales the
@@ -152,7 +152,7 @@ __global__ void __launch_bounds__(S_THREADS, 1) gemm_stream_kernel(const __grid_
                 tma_load_2d(dst + b * BOX, &wmap, k, row, fb);
                 if (SETS == 2) tma_load_2d(dst + S_W_BYTES + b * BOX, &wmap, k, M + row, fb);
             }
-            if (what & 2) tma_load_2d(dst + SETS * S_W_BYTES + b * S_XBOX, &xmap, k, group_rows ? row / group_rows * N : 0, fb);
+            if (what & 2) tma_load_2d(dst + SETS * S_W_BYTES + b * S_XBOX, &xmap, k, EPI == 6 ? row / group_rows * N : 0, fb);
         }
     };
     StreamWalk pw(range);                                             // the producer's place (thread 0 only)
@@ -483,7 +483,7 @@ static int stream_launch_th(const void* act, const void* W, void* out, int N, in
     if (grid > T) grid = T;
     const cudaError_t e = mb_launch(mb_pdl != 0, gemm_stream_kernel<EPI, SCALED, TH>, dim3((unsigned)grid), dim3(S_THREADS),
                                     SH::BYTES, st, wmap, xmap, out, N, M, K, tiles, workspace, counters, nrm, bias, after, err,
-                                    groups > 1 ? M / groups : 0);
+                                    M / groups);
     return e == cudaSuccess ? 0 : (int)e;
 }
 
@@ -531,7 +531,7 @@ MB_API int mb_gemm_stream(const void* act, const float* ssq, float eps, const vo
 // (M / groups a multiple of 128), out (N, M) bf16: the columns of group g come from act[g].
 MB_API int mb_gemm_stream_groups(const void* act, const void* W, void* out, int N, int M, int K, int groups, float* workspace,
                                  int* counters, int* err, cudaStream_t st) {
-    return stream_launch<0, false>(act, W, out, N, M, K, workspace, counters, StreamNorm{}, nullptr, StreamAfter{}, err, st,
+    return stream_launch<6, false>(act, W, out, N, M, K, workspace, counters, StreamNorm{}, nullptr, StreamAfter{}, err, st,
                                    groups);
 }
 
